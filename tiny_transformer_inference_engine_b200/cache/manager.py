@@ -20,8 +20,9 @@ step) tokens: its share stops growing there and the rest goes to the other group
 
 Pages go back to the allocator when the request is released (finished or preempted)
 and, for a windowed or chunked group, as soon as every position of the page lies before the
-window (or the chunk) of the next token to run; a freed page's table entry becomes 0 (scratch) and is
-never read because the kernels start at the window's (the chunk's) first key.  Freed pages are used
+window (or the chunk) of the next token to run - except the pages of the first tokens that a window keeps; a freed page's
+table entry becomes 0 (scratch) and what it would hold is never visible: the kernels walk the kept keys and those from the
+window's (the chunk's) first key on.  Freed pages are used
 again at once (LIFO) and are not cleared: reads are bounded by the request's length.
 
 State slots: ``max_slots`` ids; a request takes one at admission and gives it back at
@@ -81,6 +82,16 @@ class CacheGroup:
         first_key = max(0, start - self.window + 1)
         return first_key // self.page_size
 
+    @property
+    def kept_pages(self) -> int:
+        """Leading pages that are never given back while the request lives: those of the first tokens a window keeps."""
+        return pages_for(self.need.keep_first, self.page_size) if self.need.window is not None else 0
+
+    def needed_pages(self, start: int, last: int):
+        """Logical pages below ``last`` that tokens at positions >= start can read, in order: the kept ones and those of the window."""
+        first = self.first_needed_page(start)
+        return [*range(0, min(self.kept_pages, first, last)), *range(first, last)]
+
     def bytes_per_page(self, elem_size: int) -> int:
         # models/model_config.py:84-88, per group
         return self.need.planes * len(self.entries) * self.page_size * self.need.num_kv_heads * self.need.head_dim * elem_size
@@ -91,7 +102,7 @@ class CacheGroup:
         whole = pages_for(num_tokens, self.page_size)
         if self.reach is None or max_step_tokens is None:
             return whole
-        return min(whole, pages_for(self.reach + max_step_tokens - 1, self.page_size) + 1)
+        return min(whole, self.kept_pages + pages_for(self.reach + max_step_tokens - 1, self.page_size) + 1)
 
 
 class CacheManager:
@@ -195,8 +206,8 @@ class CacheManager:
                 plan.append(([], list(range(len(table), last)), last))
                 continue
             first = g.first_needed_page(start)
-            to_free = [(i, p) for i, p in enumerate(table[:first]) if p != 0]
-            to_fill = [i for i in range(first, last) if i >= len(table) or table[i] == 0]
+            to_free = [(i, p) for i, p in enumerate(table[:first]) if p != 0 and i >= g.kept_pages]
+            to_fill = [i for i in g.needed_pages(start, last) if i >= len(table) or table[i] == 0]
             plan.append((to_free, to_fill, last))
         return plan
 

@@ -29,7 +29,7 @@ struct MmaParams {
     const int* qsl; const int* seq_lens;
     __nv_bfloat16* out;
     int num_seqs, Hq, Hkv;
-    float scale_log2; int window, chunk;
+    float scale_log2; int window, chunk, keep;
     float cap_in, cap_out;              // score softcap: raw score s becomes cap_out * tanh(s * cap_in) (cap_in 0: none)
     int row_tiles, num_splits, split_len;
     float* ws_o; float* ws_ml;
@@ -103,14 +103,10 @@ paged_attn_mma_kernel(const MmaParams p) {
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 
     const int tok_lo = row0 / G, tok_hi = (min(nrows, row0 + BM) - 1) / G;
-    int k_hi = ctx + tok_hi + 1;
-    int k_lo = first_visible_key(ctx + tok_lo, p.window, p.chunk);
-    if (p.num_splits > 1) {
-        const int piece = piece_len(kv_len, p.num_splits, p.split_len, BN);
-        k_lo = max(k_lo, split * piece);
-        k_hi = min(k_hi, (split + 1) * piece);
-    }
-    k_lo = k_lo / BN * BN;                                                          // tiles start on multiples of BN
+    const int k_hi = ctx + tok_hi + 1;
+    const KeySpan span = visible_span(ctx + tok_lo, k_hi, p.window, p.chunk, p.keep, BN);      // tiles start on multiples of BN
+    int v_lo, v_hi;                                                                 // this CTA's piece, as indices into the span
+    span_piece(span, kv_len, p.window > 0 || p.chunk > 0, split, p.num_splits, p.split_len, BN, v_lo, v_hi);
 
     // the two rows of this thread
     int rpos[2], rlo[2]; bool rvalid[2]; int rrow[2];
@@ -140,7 +136,7 @@ paged_attn_mma_kernel(const MmaParams p) {
 #pragma unroll
     for (int i = 0; i < D / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
 
-    const int ntiles = k_lo < k_hi ? (k_hi - k_lo + BN - 1) / BN : 0;
+    const int ntiles = v_lo < v_hi ? (v_hi - v_lo + BN - 1) / BN : 0;
     const int* table = p.block_table + (size_t)seq * p.table_width;
 
     auto fill_rowoff = [&](int stage, int kt) {
@@ -178,7 +174,7 @@ paged_attn_mma_kernel(const MmaParams p) {
             const __nv_bfloat16* src = p.q + (size_t)(q0 + tok) * p.q_stride + (size_t)(kvh * G + g) * D + part * 8;
             cp_async16(Qs + r * LDS + part * 8, ok ? src : p.q, ok);
         }
-        fill_rowoff(0, k_lo);
+        fill_rowoff(0, span.key(v_lo));
         __syncthreads();
         issue_tile(0);
         cp_async_commit();
@@ -186,9 +182,9 @@ paged_attn_mma_kernel(const MmaParams p) {
 
     unsigned qf[D / 16][4];
     for (int t = 0; t < ntiles; ++t) {
-        const int stage = STAGES == 2 ? (t & 1) : 0, kt = k_lo + t * BN;
+        const int stage = STAGES == 2 ? (t & 1) : 0, kt = span.key(v_lo + t * BN);
         if (STAGES == 2) {
-            if (t + 1 < ntiles) fill_rowoff(stage ^ 1, kt + BN);
+            if (t + 1 < ntiles) fill_rowoff(stage ^ 1, span.key(v_lo + (t + 1) * BN));
             __syncthreads();                       // row offsets visible; everyone is done with the other stage
             if (t + 1 < ntiles) issue_tile(stage ^ 1);
             cp_async_commit();
@@ -209,7 +205,7 @@ paged_attn_mma_kernel(const MmaParams p) {
             for (int ks = 0; ks < D / 16; ++ks)
                 ldmatrix_x4(qf[ks], Qs + (warp * 16 + (lane & 7) + 8 * ((lane >> 3) & 1)) * LDS + ks * 16 + 8 * (lane >> 4));
         }
-        const bool needed = warp_active && kt <= wpos_hi && kt + BN > wkey_lo;
+        const bool needed = warp_active && kt <= wpos_hi && (kt + BN > wkey_lo || kt < p.keep);
         if (needed) {
             const __nv_bfloat16* kb = Ks + stage * BN * LDS;
             const __nv_bfloat16* vb = Vs + stage * BN * LDS;
@@ -239,7 +235,7 @@ paged_attn_mma_kernel(const MmaParams p) {
                     if (p.cap_in != 0.f) v = p.cap_out * tanh_ex2(v * p.cap_in);
                     if (!full) {
                         const int key = kt + i * 8 + 2 * (lane & 3) + (e & 1);
-                        if (!(rvalid[h] && key <= rpos[h] && key >= rlo[h] && key < k_hi)) v = -INFINITY;
+                        if (!(rvalid[h] && key <= rpos[h] && (key >= rlo[h] || key < p.keep) && key < k_hi)) v = -INFINITY;
                     }
                     s[i][e] = v;
                     mx[h] = fmaxf(mx[h], v);
@@ -410,11 +406,9 @@ paged_attn_cluster_kernel(const MmaParams p) {
     const int ctx = kv_len - q_len;
 
     const int tok_lo = row0 / G, tok_hi = (min(nrows, row0 + BM) - 1) / G;
-    int k_hi = ctx + tok_hi + 1;
-    int k_lo = first_visible_key(ctx + tok_lo, p.window, p.chunk);
-    k_lo = max(k_lo, (int)rank * p.split_len);
-    k_hi = min(k_hi, ((int)rank + 1) * p.split_len);
-    k_lo = k_lo / BN * BN;
+    const int k_hi = ctx + tok_hi + 1;
+    const KeySpan span = visible_span(ctx + tok_lo, k_hi, p.window, p.chunk, p.keep, BN);
+    const int v_lo = (int)rank * p.split_len, v_hi = min(span.total, v_lo + p.split_len);      // this CTA's piece, as indices into the span
 
     int rpos[2], rlo[2]; bool rvalid[2];
 #pragma unroll
@@ -435,7 +429,8 @@ paged_attn_cluster_kernel(const MmaParams p) {
 #pragma unroll
     for (int i = 0; i < D / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
 
-    const int kt0 = k_lo + kg * BN;                                                // this group's first tile
+    const int vt0 = v_lo + kg * BN;                                                // this group's first tile
+    const int kt0 = span.key(vt0);
     // this warp's 16 query rows straight into mma A fragments (4-byte loads; no shared memory, no barrier):
     // fragment registers 0,1 hold columns 2q, 2q+1 of rows g and g+8, registers 2,3 the same 8 columns on
     unsigned qf[D / 16][4];
@@ -447,7 +442,7 @@ paged_attn_cluster_kernel(const MmaParams p) {
             const int tok = rvalid[h] ? row / G : 0, g = rvalid[h] ? row - tok * G : 0;
             qrow[h] = p.q + (size_t)(q0 + tok) * p.q_stride + (size_t)(kvh * G + g) * D + 2 * (lane & 3);
         }
-        const bool any_keys = kt0 < k_hi;
+        const bool any_keys = vt0 < v_hi;
 #pragma unroll
         for (int ks = 0; ks < D / 16; ++ks)
 #pragma unroll
@@ -489,18 +484,18 @@ paged_attn_cluster_kernel(const MmaParams p) {
     // Keys and values are separate copy groups: the next tile's keys are asked for as soon as this tile's
     // scores are done, its values after the second product, so most of their latency hides behind arithmetic.
     unsigned off_cur[2], off_next[2] = {NO_ROW, NO_ROW};
-    if (kt0 < k_hi) {
+    if (vt0 < v_hi) {
         row_offsets(off_cur, kt0, kt0 == kt_guess ? page_guess : nullptr);
         issue(kb, p.k_pages, off_cur);
         issue(vb, p.v_pages, off_cur);
     }
-    for (int kt = kt0; kt < k_hi; kt += KG * BN) {
-        const int kt_next = kt + KG * BN;
-        const bool more = kt_next < k_hi;
-        if (more) row_offsets(off_next, kt_next, nullptr);      // (its page loads overlap the wait below)
+    for (int vt = vt0; vt < v_hi; vt += KG * BN) {
+        const int kt = span.key(vt);
+        const bool more = vt + KG * BN < v_hi;
+        if (more) row_offsets(off_next, span.key(vt + KG * BN), nullptr);      // (its page loads overlap the wait below)
         cp_async_wait<1>();                                     // this tile's keys (its values may still be on their way)
         group_sync();
-        const bool needed = warp_active && kt <= wpos_hi && kt + BN > wkey_lo;
+        const bool needed = warp_active && kt <= wpos_hi && (kt + BN > wkey_lo || kt < p.keep);
         float s[BN / 8][4];
         if (needed) {
 #pragma unroll
@@ -531,7 +526,7 @@ paged_attn_cluster_kernel(const MmaParams p) {
                     if (p.cap_in != 0.f) v = p.cap_out * tanh_ex2(v * p.cap_in);
                     if (!full) {
                         const int key = kt + i * 8 + 2 * (lane & 3) + (e & 1);
-                        if (!(rvalid[h] && key <= rpos[h] && key >= rlo[h] && key < k_hi)) v = -INFINITY;
+                        if (!(rvalid[h] && key <= rpos[h] && (key >= rlo[h] || key < p.keep) && key < k_hi)) v = -INFINITY;
                     }
                     s[i][e] = v;
                     mx[h] = fmaxf(mx[h], v);
@@ -814,7 +809,7 @@ extern "C" int ttie_paged_attention_mma(const void* q, long long q_stride, const
 extern "C" int ttie_paged_attention_mma_weights(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
                                                 const int* block_table, int table_width, int page_size, const int* qsl,
                                                 const int* seq_lens, void* out, int T, int num_seqs, int Hq, int Hkv, int D,
-                                                int max_q_len, float scale, float softcap, int window, int chunk, int num_splits, int split_len,
+                                                int max_q_len, float scale, float softcap, int window, int chunk, int keep, int num_splits, int split_len,
                                                 float* scratch, int form, int weights, const float* head_bias, void* stream);
 
 extern "C" int ttie_paged_attention_mma_form(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
@@ -823,14 +818,14 @@ extern "C" int ttie_paged_attention_mma_form(const void* q, long long q_stride, 
                                              int max_q_len, float scale, float softcap, int window, int chunk, int num_splits, int split_len,
                                              float* scratch, int form, void* stream) {
     return ttie_paged_attention_mma_weights(q, q_stride, k_pages, v_pages, block_table, table_width, page_size, qsl, seq_lens, out, T, num_seqs,
-                                            Hq, Hkv, D, max_q_len, scale, softcap, window, chunk, num_splits, split_len, scratch, form, 0, nullptr,
+                                            Hq, Hkv, D, max_q_len, scale, softcap, window, chunk, 0, num_splits, split_len, scratch, form, 0, nullptr,
                                             stream);
 }
 
 extern "C" int ttie_paged_attention_mma_weights(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
                                                 const int* block_table, int table_width, int page_size, const int* qsl,
                                                 const int* seq_lens, void* out, int T, int num_seqs, int Hq, int Hkv, int D,
-                                                int max_q_len, float scale, float softcap, int window, int chunk, int num_splits, int split_len,
+                                                int max_q_len, float scale, float softcap, int window, int chunk, int keep, int num_splits, int split_len,
                                                 float* scratch, int form, int weights, const float* head_bias, void* stream) {
     if (T <= 0 || num_seqs <= 0) return 0;
     if (weights != 0 && weights != 1) TTIE_FAIL("paged_attention_mma: unknown kind of weights %d", weights);
@@ -849,7 +844,7 @@ extern "C" int ttie_paged_attention_mma_weights(const void* q, long long q_strid
     p.block_table = block_table; p.table_width = table_width; p.page_size = page_size;
     p.qsl = qsl; p.seq_lens = seq_lens; p.out = (__nv_bfloat16*)out;
     p.num_seqs = num_seqs; p.Hq = Hq; p.Hkv = Hkv;
-    p.scale_log2 = scale * 1.4426950408889634f; p.window = window; p.chunk = chunk;
+    p.scale_log2 = scale * 1.4426950408889634f; p.window = window; p.chunk = chunk; p.keep = window > 0 ? keep : 0;
     p.cap_in = softcap > 0.f ? scale / softcap : 0.f; p.cap_out = softcap > 0.f ? softcap / scale : 0.f;
     p.num_splits = num_splits; p.split_len = split_len;
     p.sigmoid = weights; p.head_bias = head_bias;
@@ -857,7 +852,7 @@ extern "C" int ttie_paged_attention_mma_weights(const void* q, long long q_strid
     const int rows = max_q_len * (Hq / Hkv);
     if (form == 2 || form == 4) {
         if (num_splits > 1 && (split_len <= 0 || split_len % BN)) TTIE_FAIL("paged_attention_mma: the split length must be a multiple of %d", BN);
-        if (num_splits == 1) p.split_len = 1 << 30;
+        if (num_splits == 1) p.split_len = 1 << 29;
         const int tile_rows = ttie_attn_cluster_tile_rows(max_q_len, Hq, Hkv);
         p.row_tiles = ceil_div(rows, tile_rows);
         if ((long long)num_seqs * Hkv * p.row_tiles > 2147483647LL) TTIE_FAIL("paged_attention_mma: grid too large");

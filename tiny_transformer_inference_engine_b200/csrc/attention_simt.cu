@@ -18,6 +18,11 @@
 // Sigmoid weights (instead of a softmax): the weight of a visible key is sigmoid(score + bias of the row's head), weights are
 // not normalised over keys, so a row's output is a plain sum and the pieces of a cut key range simply add: each piece leaves
 // (maximum 0, sum 1 / pieces) beside its partial output, with which the merge kernels' formula is that plain sum.
+//
+// Joint rows (paged_attn_joint_kernel): all query heads score against ONE key row per token - the rows of all kv heads side by
+// side -, each with a query row as long as that, while the values stay those of the head's own kv head: columns
+// vh * Dv .. of a value row that holds all kv heads' values.  Score rows mixed over heads take this form (head_mix.cu).  The
+// key row may be long (16 kv heads of 64: 1,024), so scores are accumulated over pieces of JC of its columns.
 #include "common.cuh"
 #include <math.h>
 using namespace ttie;
@@ -32,7 +37,7 @@ struct AttnParams {
     const int* qsl; const int* seq_lens;
     void* out;
     int num_seqs, Hq, Hkv, D;
-    float scale; int window, chunk;
+    float scale; int window, chunk, keep;      // keep: first tokens of the sequence that stay visible behind a window
     float softcap;                 // > 0: scores pass cap * tanh(score / cap) before mask and softmax
     int sigmoid;                   // 1: a visible key weighs sigmoid(score + head_bias[head]); no softmax
     const float* head_bias;        // [Hq] or null (sigmoid weights only)
@@ -72,13 +77,10 @@ paged_attn_simt_kernel(const AttnParams p) {
 
     const int tok_lo = row0 / G;
     const int tok_hi = (min(nrows, row0 + ROWS) - 1) / G;
-    int k_hi = ctx + tok_hi + 1;
-    int k_lo = first_visible_key(ctx + tok_lo, p.window, p.chunk);
-    if (p.num_splits > 1) {
-        const int piece = piece_len(kv_len, p.num_splits, p.split_len, BK);
-        k_lo = max(k_lo, split * piece);
-        k_hi = min(k_hi, (split + 1) * piece);
-    }
+    const int k_hi = ctx + tok_hi + 1;
+    const KeySpan span = visible_span(ctx + tok_lo, k_hi, p.window, p.chunk, p.keep, BK);
+    int v_lo, v_hi;                                                  // this CTA's piece, as indices into the span
+    span_piece(span, kv_len, p.window > 0 || p.chunk > 0, split, p.num_splits, p.split_len, BK, v_lo, v_hi);
 
     // per-row state of this warp's rows
     float m[RPW], l[RPW], o[RPW][DPL];
@@ -98,7 +100,7 @@ paged_attn_simt_kernel(const AttnParams p) {
         for (int i = 0; i < DPL; ++i) o[r][i] = 0.f;
     }
 
-    if (k_lo < k_hi) {
+    if (v_lo < v_hi) {
         const T* qp = (const T*)p.q;
         for (int idx = threadIdx.x; idx < ROWS * D; idx += blockDim.x) {
             const int r = idx / D, d = idx - r * D;
@@ -114,7 +116,8 @@ paged_attn_simt_kernel(const AttnParams p) {
         const T* vp = (const T*)p.v_pages;
         const int* table = p.block_table + (size_t)seq * p.table_width;
 
-        for (int kt = k_lo; kt < k_hi; kt += BK) {
+        for (int vt = v_lo; vt < v_hi; vt += BK) {
+            const int kt = span.key(vt);
             __syncthreads();
             // four consecutive elements of a key and of a value per step (head sizes are multiples of 4): one page look-up
             // and one 16-byte (float32) or 8-byte (bfloat16) load of each
@@ -152,7 +155,7 @@ paged_attn_simt_kernel(const AttnParams p) {
             float pr[RPW];
 #pragma unroll
             for (int r = 0; r < RPW; ++r) {
-                const bool vis = valid[r] && key < k_hi && key <= pos[r] && key >= lo[r];
+                const bool vis = valid[r] && key < k_hi && key <= pos[r] && (key >= lo[r] || key < p.keep);
                 float sv = s[r] * p.scale;
                 if (p.softcap > 0.f) sv = p.softcap * tanhf(sv / p.softcap);
                 if (p.sigmoid) { pr[r] = vis ? 1.0f / (1.0f + expf(-(sv + hb[r]))) : 0.f; continue; }
@@ -408,7 +411,236 @@ int dispatch(const AttnParams& p, int T_tokens, cudaStream_t s) {
     }
     TTIE_FAIL("paged_attention: head size %d not supported (multiples of 4 up to 512)", p.D);
 }
+// ---- joint rows: any number of kv heads, key row width W (a multiple of 4), value size Dv (up to 512), float32 arithmetic
+constexpr int JC = 128;                     // columns of the key rows staged at a time
+
+struct JointParams {
+    const void* q;                          // [T, H, W]
+    const void* k_pages; const void* v_pages;                        // [pages, page_size, W] each
+    const int* block_table; int table_width; int page_size;
+    const int* qsl; const int* seq_lens;
+    void* out;                              // [T, H, Dv]
+    int num_seqs, H, G, W, Dv;              // G: kv heads (value groups)
+    float scale; int window, chunk, keep;
+    int row_tiles, num_splits, split_len;
+    float* ws_o; float* ws_ml;              // [T*H, num_splits, Dv] and [T*H, num_splits, 2]
+};
+
+template <typename T, int DPL, int RW>
+__global__ void __launch_bounds__(WARPS * 32)
+paged_attn_joint_kernel(const JointParams p) {
+    constexpr int NROWS = WARPS * RW, KS = JC + 4;
+    extern __shared__ __align__(16) float smem[];
+    TTIE_PDL_ENTRY();
+    const int W = p.W, Dv = p.Dv, per = p.H / p.G;
+    float* Qs = smem;                       // [NROWS][W]
+    float* Ks = Qs + NROWS * W;             // [BK][JC + 4]
+    float* Vs = Ks + BK * KS;               // [BK][Dv]
+
+    int tile = blockIdx.x;
+    const int split = blockIdx.y;
+    const int rt = tile % p.row_tiles; tile /= p.row_tiles;
+    const int vh = tile % p.G;
+    const int seq = tile / p.G;
+    const int q0 = p.qsl[seq], q_len = p.qsl[seq + 1] - q0, kv_len = p.seq_lens[seq];
+    const int nrows = q_len * per;
+    const int row0 = rt * NROWS;
+    if (row0 >= nrows) return;
+    const int ctx = kv_len - q_len;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+
+    const int tok_lo = row0 / per;
+    const int tok_hi = (min(nrows, row0 + NROWS) - 1) / per;
+    const int k_hi = ctx + tok_hi + 1;
+    const KeySpan span = visible_span(ctx + tok_lo, k_hi, p.window, p.chunk, p.keep, BK);
+    int v_lo, v_hi;
+    span_piece(span, kv_len, p.window > 0 || p.chunk > 0, split, p.num_splits, p.split_len, BK, v_lo, v_hi);
+
+    float m[RW], l[RW], o[RW][DPL];
+    int pos[RW], lo[RW];
+    bool valid[RW];
+#pragma unroll
+    for (int r = 0; r < RW; ++r) {
+        const int row = row0 + warp * RW + r;
+        valid[r] = row < nrows;
+        pos[r] = ctx + (valid[r] ? row / per : 0);
+        lo[r] = first_visible_key(pos[r], p.window, p.chunk);
+        m[r] = -INFINITY; l[r] = 0.f;
+#pragma unroll
+        for (int i = 0; i < DPL; ++i) o[r][i] = 0.f;
+    }
+
+    if (v_lo < v_hi) {
+        const T* qp = (const T*)p.q;
+        const int W4 = W >> 2;
+        for (int idx = threadIdx.x; idx < NROWS * W4; idx += blockDim.x) {
+            const int r = idx / W4, d = (idx - r * W4) << 2;
+            const int row = row0 + r;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (row < nrows) {
+                const int tok = row / per, g = row - tok * per;
+                v = load4(qp + ((size_t)(q0 + tok) * p.H + vh * per + g) * W + d);
+            }
+            *reinterpret_cast<float4*>(Qs + r * W + d) = v;
+        }
+        const T* kp = (const T*)p.k_pages;
+        const T* vp = (const T*)p.v_pages;
+        const int* table = p.block_table + (size_t)seq * p.table_width;
+        auto row_of = [&](int key) -> size_t {                       // (a table that is too short: the scratch page, not a wild read)
+            const int pg = key / p.page_size;
+            const int page = pg < p.table_width ? table[pg] : 0;
+            return ((size_t)page * p.page_size + (key - pg * p.page_size)) * W;
+        };
+
+        for (int vt = v_lo; vt < v_hi; vt += BK) {
+            const int kt = span.key(vt);
+            const int key = kt + lane;
+            float s[RW];
+#pragma unroll
+            for (int r = 0; r < RW; ++r) s[r] = 0.f;
+            for (int c0 = 0; c0 < W; c0 += JC) {
+                const int nc = min(JC, W - c0);
+                __syncthreads();                                     // everyone is done with the last piece (and with the last tile's values)
+                for (int idx = threadIdx.x; idx < BK * (nc >> 2); idx += blockDim.x) {
+                    const int j = idx / (nc >> 2), d = (idx - j * (nc >> 2)) << 2;
+                    float4 kval = make_float4(0.f, 0.f, 0.f, 0.f);
+                    if (kt + j < k_hi) kval = load4(kp + row_of(kt + j) + c0 + d);
+                    *reinterpret_cast<float4*>(Ks + j * KS + d) = kval;
+                }
+                if (c0 == 0)
+                    for (int idx = threadIdx.x; idx < BK * Dv; idx += blockDim.x) {
+                        const int j = idx / Dv, d = idx - j * Dv;
+                        Vs[idx] = kt + j < k_hi ? to_f32<T>(vp[row_of(kt + j) + (size_t)vh * Dv + d]) : 0.f;
+                    }
+                __syncthreads();
+                const float4* k4 = reinterpret_cast<const float4*>(Ks + lane * KS);
+                for (int d4 = 0; d4 < (nc >> 2); ++d4) {
+                    const float4 kv = k4[d4];
+#pragma unroll
+                    for (int r = 0; r < RW; ++r) {
+                        const float4 qv = *reinterpret_cast<const float4*>(Qs + (warp * RW + r) * W + c0 + 4 * d4);
+                        s[r] = fmaf(qv.x, kv.x, s[r]); s[r] = fmaf(qv.y, kv.y, s[r]);
+                        s[r] = fmaf(qv.z, kv.z, s[r]); s[r] = fmaf(qv.w, kv.w, s[r]);
+                    }
+                }
+            }
+            float pr[RW];
+#pragma unroll
+            for (int r = 0; r < RW; ++r) {
+                const bool vis = valid[r] && key < k_hi && key <= pos[r] && (key >= lo[r] || key < p.keep);
+                const float sc = vis ? s[r] * p.scale : -INFINITY;
+                const float m_new = fmaxf(m[r], warp_max(sc));
+                const float alpha = (m[r] == -INFINITY) ? 0.f : expf(m[r] - m_new);
+                pr[r] = vis ? expf(sc - m_new) : 0.f;
+                l[r] = l[r] * alpha + warp_sum(pr[r]);
+                m[r] = m_new;
+#pragma unroll
+                for (int i = 0; i < DPL; ++i) o[r][i] *= alpha;
+            }
+            const int nk = min(BK, k_hi - kt);
+            for (int j = 0; j < nk; ++j) {
+                float vv[DPL];
+#pragma unroll
+                for (int i = 0; i < DPL; ++i) vv[i] = lane + 32 * i < Dv ? Vs[j * Dv + lane + 32 * i] : 0.f;
+#pragma unroll
+                for (int r = 0; r < RW; ++r) {
+                    const float pj = __shfl_sync(0xffffffffu, pr[r], j);
+#pragma unroll
+                    for (int i = 0; i < DPL; ++i) o[r][i] = fmaf(pj, vv[i], o[r][i]);
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < RW; ++r) {
+        if (!valid[r]) continue;
+        const int row = row0 + warp * RW + r;
+        const int tok = row / per, g = row - tok * per;
+        const size_t grow = (size_t)(q0 + tok) * p.H + vh * per + g;
+        const bool whole = p.num_splits == 1;
+        const float inv = whole ? (l[r] > 0.f ? 1.f / l[r] : 0.f) : 1.f;
+#pragma unroll
+        for (int i = 0; i < DPL; ++i) {
+            const int d = lane + 32 * i;
+            if (d >= Dv) continue;
+            if (whole) ((T*)p.out)[grow * Dv + d] = from_f32<T>(o[r][i] * inv);
+            else p.ws_o[(grow * p.num_splits + split) * Dv + d] = o[r][i];
+        }
+        if (!whole && lane == 0) {
+            float* ml = p.ws_ml + (grow * p.num_splits + split) * 2;
+            ml[0] = m[r]; ml[1] = l[r];
+        }
+    }
+}
+
+constexpr int JOINT_SMEM = 220 * 1024;
+size_t joint_smem(int W, int Dv, int rows) { return ((size_t)rows * W + (size_t)BK * (JC + 4) + (size_t)BK * Dv) * sizeof(float); }
+// query rows per warp: 4, or 1 where four rows of the joint width do not fit shared memory; 0: not even one
+int joint_rows_per_warp(int W, int Dv) {
+    return joint_smem(W, Dv, 4 * WARPS) <= JOINT_SMEM ? 4 : joint_smem(W, Dv, WARPS) <= JOINT_SMEM ? 1 : 0;
+}
+
+template <typename T, int DPL, int RW>
+int launch_joint(const JointParams& p, int T_tokens, cudaStream_t s) {
+    const size_t smem = joint_smem(p.W, p.Dv, RW * WARPS);
+    auto k = paged_attn_joint_kernel<T, DPL, RW>;
+    if (smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) TTIE_FAIL("paged_attention_joint: %zu bytes of shared memory refused: %s", smem, cudaGetErrorString(e));
+    }
+    TTIE_LAUNCH(k, dim3(p.num_seqs * p.G * p.row_tiles, p.num_splits), WARPS * 32, smem, s, p);
+    TTIE_CHECK_LAUNCH("paged_attention_joint");
+    if (p.num_splits > 1) {
+        attn_merge_kernel<T><<<T_tokens * p.H, MERGE_GROUPS * (p.Dv >= 128 ? 128 : 64), (p.num_splits + MERGE_GROUPS * p.Dv) * sizeof(float), s>>>(
+            p.ws_o, p.ws_ml, (T*)p.out, p.num_splits, p.Dv);
+        TTIE_CHECK_LAUNCH("attention merge");
+    }
+    return 0;
+}
+template <typename T, int RW>
+int dispatch_joint(const JointParams& p, int T_tokens, cudaStream_t s) {
+    const int n = (p.Dv + 31) / 32;
+    if (n <= 1) return launch_joint<T, 1, RW>(p, T_tokens, s);
+    if (n <= 2) return launch_joint<T, 2, RW>(p, T_tokens, s);
+    if (n <= 4) return launch_joint<T, 4, RW>(p, T_tokens, s);
+    if (n <= 8) return launch_joint<T, 8, RW>(p, T_tokens, s);
+    return launch_joint<T, 16, RW>(p, T_tokens, s);
+}
 }  // namespace
+
+// Query rows per CTA of the joint-row kernel for these sizes; 0: it does not take them.
+extern "C" int ttie_attn_joint_tile_rows(int W, int Dv) {
+    return (W <= 0 || W % 4 || Dv <= 0 || Dv > 512) ? 0 : WARPS * joint_rows_per_warp(W, Dv);
+}
+
+// q [T, H, W]; pages [pages, page_size, W]; out [T, H, Dv]; scratch: T*H*num_splits*(Dv + 2) floats where num_splits > 1
+extern "C" int ttie_paged_attention_joint(const void* q, const void* k_pages, const void* v_pages, const int* block_table, int table_width,
+                                          int page_size, const int* qsl, const int* seq_lens, void* out, int T, int num_seqs, int H, int G,
+                                          int W, int Dv, int max_q_len, float scale, int window, int chunk, int keep, int num_splits,
+                                          int split_len, float* scratch, int dtype, void* stream) {
+    if (T <= 0 || num_seqs <= 0) return 0;
+    if (G <= 0 || H % G) TTIE_FAIL("paged_attention_joint: %d heads are not a multiple of %d kv heads", H, G);
+    const int tile_rows = ttie_attn_joint_tile_rows(W, Dv);
+    if (!tile_rows || (long long)G * Dv > W)
+        TTIE_FAIL("paged_attention_joint: rows of %d values with %d x %d value columns are not supported", W, G, Dv);
+    if (page_size <= 0) TTIE_FAIL("paged_attention_joint: page size %d", page_size);
+    if (num_splits < 1) num_splits = 1;
+    if (num_splits > 1 && (split_len <= 0 || split_len % BK || !scratch)) TTIE_FAIL("paged_attention_joint: splits need scratch and a split length that is a multiple of %d", BK);
+    if (num_splits > 65535) TTIE_FAIL("paged_attention_joint: too many splits (%d)", num_splits);
+    JointParams p;
+    p.q = q; p.k_pages = k_pages; p.v_pages = v_pages; p.block_table = block_table; p.table_width = table_width; p.page_size = page_size;
+    p.qsl = qsl; p.seq_lens = seq_lens; p.out = out; p.num_seqs = num_seqs; p.H = H; p.G = G; p.W = W; p.Dv = Dv;
+    p.scale = scale; p.window = window; p.chunk = chunk; p.keep = window > 0 ? keep : 0;
+    p.row_tiles = ceil_div(max_q_len * (H / G), tile_rows);
+    p.num_splits = num_splits; p.split_len = split_len;
+    p.ws_o = scratch; p.ws_ml = scratch ? scratch + (size_t)T * H * num_splits * Dv : nullptr;
+    if ((long long)num_seqs * G * p.row_tiles > 2147483647LL) TTIE_FAIL("paged_attention_joint: grid too large");
+    cudaStream_t s = (cudaStream_t)stream;
+    const bool wide = joint_rows_per_warp(W, Dv) == 1;
+    if (dtype == kF32) return wide ? dispatch_joint<float, 1>(p, T, s) : dispatch_joint<float, 4>(p, T, s);
+    if (dtype == kBF16) return wide ? dispatch_joint<__nv_bfloat16, 1>(p, T, s) : dispatch_joint<__nv_bfloat16, 4>(p, T, s);
+    TTIE_FAIL("paged_attention_joint: unknown dtype %d", dtype);
+}
 
 // Scratch floats needed for `num_splits` splits: the caller allocates ws_o and ws_ml.
 extern "C" long long ttie_attn_scratch_floats(int T, int Hq, int D, int num_splits) {
@@ -419,7 +651,7 @@ extern "C" long long ttie_attn_scratch_floats(int T, int Hq, int D, int num_spli
 extern "C" int ttie_paged_attention_weights(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
                                             const int* block_table, int table_width, int page_size, const int* qsl,
                                             const int* seq_lens, void* out, int T, int num_seqs, int Hq, int Hkv, int D,
-                                            int max_q_len, float scale, float softcap, int window, int chunk, int num_splits, int split_len,
+                                            int max_q_len, float scale, float softcap, int window, int chunk, int keep, int num_splits, int split_len,
                                             float* scratch, int dtype, int weights, const float* head_bias, void* stream);
 
 extern "C" int ttie_paged_attention(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
@@ -428,14 +660,14 @@ extern "C" int ttie_paged_attention(const void* q, long long q_stride, const voi
                                     int max_q_len, float scale, float softcap, int window, int chunk, int num_splits, int split_len,
                                     float* scratch, int dtype, void* stream) {
     return ttie_paged_attention_weights(q, q_stride, k_pages, v_pages, block_table, table_width, page_size, qsl, seq_lens, out, T, num_seqs,
-                                        Hq, Hkv, D, max_q_len, scale, softcap, window, chunk, num_splits, split_len, scratch, dtype, 0, nullptr,
+                                        Hq, Hkv, D, max_q_len, scale, softcap, window, chunk, 0, num_splits, split_len, scratch, dtype, 0, nullptr,
                                         stream);
 }
 
 extern "C" int ttie_paged_attention_weights(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
                                             const int* block_table, int table_width, int page_size, const int* qsl,
                                             const int* seq_lens, void* out, int T, int num_seqs, int Hq, int Hkv, int D,
-                                            int max_q_len, float scale, float softcap, int window, int chunk, int num_splits, int split_len,
+                                            int max_q_len, float scale, float softcap, int window, int chunk, int keep, int num_splits, int split_len,
                                             float* scratch, int dtype, int weights, const float* head_bias, void* stream) {
     if (T <= 0 || num_seqs <= 0) return 0;
     if (D % 4 || D > 512 || D <= 0) TTIE_FAIL("paged_attention: head size %d not supported (multiples of 4 up to 512)", D);
@@ -447,7 +679,7 @@ extern "C" int ttie_paged_attention_weights(const void* q, long long q_stride, c
     p.q = q; p.q_stride = q_stride; p.k_pages = k_pages; p.v_pages = v_pages;
     p.block_table = block_table; p.table_width = table_width; p.page_size = page_size;
     p.qsl = qsl; p.seq_lens = seq_lens; p.out = out;
-    p.num_seqs = num_seqs; p.Hq = Hq; p.Hkv = Hkv; p.D = D; p.scale = scale; p.window = window; p.chunk = chunk; p.softcap = softcap;
+    p.num_seqs = num_seqs; p.Hq = Hq; p.Hkv = Hkv; p.D = D; p.scale = scale; p.window = window; p.chunk = chunk; p.keep = window > 0 ? keep : 0; p.softcap = softcap;
     if (weights != 0 && weights != 1) TTIE_FAIL("paged_attention: unknown kind of weights %d", weights);
     p.sigmoid = weights; p.head_bias = head_bias;
     const int G = Hq / Hkv;

@@ -153,7 +153,7 @@ struct AttnTcParams {
     const int* qsl; const int* seq_lens;
     __nv_bfloat16* out;
     int num_seqs, Hq, Hkv;
-    float scale_log2; int window, chunk;
+    float scale_log2; int window, chunk, keep;                   // keep: first tokens of the sequence that stay visible behind a window
     float cap_in, cap_out;                                       // score softcap: raw score s becomes cap_out * tanh(s * cap_in) (cap_in 0: none)
     int row_tiles;
     int q_rows;                                                  // rows of the query tile that are staged (a multiple of 32 that covers every request's rows)
@@ -217,16 +217,11 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
     if (row0 >= nrows) return;                                   // uniform over the CTA, before anything is allocated
     const int ctx = kv_len - q_len;
     const int tok_lo = row0 / G, tok_hi = (min(nrows, row0 + BM) - 1) / G;
-    int key_hi = ctx + tok_hi + 1;                               // exclusive
-    int key_lo = first_visible_key(ctx + tok_lo, p.window, p.chunk);
+    const KeySpan span = visible_span(ctx + tok_lo, ctx + tok_hi + 1, p.window, p.chunk, p.keep, BN);
     const int split = blockIdx.y;
-    if (p.num_splits > 1) {                                      // splits start on tile boundaries
-        const int piece = piece_len(kv_len, p.num_splits, p.split_len, BN);
-        key_lo = max(key_lo, split * piece);
-        key_hi = min(key_hi, (split + 1) * piece);
-    }
-    const int t_begin = key_lo / BN, t_end = (key_hi + BN - 1) / BN;
-    const int ntiles = t_end - t_begin;
+    int v_lo, v_hi;                                              // this CTA's piece, as indices into the span; pieces start on tile boundaries
+    span_piece(span, kv_len, p.window > 0 || p.chunk > 0, split, p.num_splits, p.split_len, BN, v_lo, v_hi);
+    const int ntiles = v_lo < v_hi ? (v_hi - v_lo + BN - 1) / BN : 0;
     const int rows_here = min(BM, nrows - row0);
     if (ntiles <= 0) {
         // (only with splits) no key of this split is visible: an empty partial result, nothing allocated.  The scratch
@@ -271,7 +266,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
             const int box_rows = ps < BN ? ps : BN, nboxes = BN / box_rows;            // at most 16 boxes per tile
             const int jt = lane / nboxes, bx = lane - jt * nboxes;
             if (jt < 2 && jt < ntiles) {
-                const int key = (t_begin + jt) * BN + bx * box_rows;
+                const int key = span.key(v_lo + jt * BN) + bx * box_rows;
                 const int pg = key / ps;
                 const int page = pg < p.table_width ? p.block_table[(size_t)seq * p.table_width + pg] : 0;
                 y_first = (page * p.Hkv + kvh) * ps + (key - pg * ps);
@@ -315,7 +310,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
         auto box_row = [&](int j) -> int {                      // first row of this lane's box of tile j in the page matrix
             int y = 0;
             if (lane < nboxes && j < ntiles) {
-                const int key = (t_begin + j) * BN + lane * box_rows;
+                const int key = span.key(v_lo + j * BN) + lane * box_rows;
                 const int pg = key / ps;
                 const int page = pg < p.table_width ? table[pg] : 0;
                 y = (page * p.Hkv + kvh) * ps + (key - pg * ps);
@@ -359,7 +354,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
         auto box_row = [&](int j) -> int {                      // first row of this lane's box of tile j in the page matrix
             int y = 0;
             if (lane < nboxes && j < ntiles) {
-                const int key = (t_begin + j) * BN + lane * box_rows;
+                const int key = span.key(v_lo + j * BN) + lane * box_rows;
                 const int pg = key / ps;
                 const int page = pg < p.table_width ? table[pg] : 0;
                 y = (page * p.Hkv + kvh) * ps + (key - pg * ps);
@@ -479,10 +474,10 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
                 ok = __all_sync(0xffffffffu, ok);
                 if (!ok) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                const int key0 = (t_begin + j) * BN;
-                // columns lo_col..hi_col of this tile are visible to the row; a tile that every row of the warp
-                // sees whole takes the path without compares
-                const int hi_col = valid ? pos - key0 : -1, lo_col = lo - key0;
+                const int key0 = span.key(v_lo + j * BN);
+                // columns lo_col..hi_col of this tile are visible to the row, and with kept first tokens the columns below
+                // keep_col; a tile that every row of the warp sees whole takes the path without compares
+                const int hi_col = valid ? pos - key0 : -1, lo_col = lo - key0, keep_col = p.keep - key0;
                 const bool tile_full = __all_sync(0xffffffffu, valid && hi_col >= BN - 1 && lo_col <= 0);
                 uint32_t sv[SC];
                 tmem_ld32(lane_addr + S_COL + sb * BN + part * SC, sv);
@@ -496,7 +491,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
 #pragma unroll
                     for (int i = 0; i < SC; ++i) {
                         const int col = part * SC + i;
-                        if (!(col <= hi_col && col >= lo_col)) sv[i] = 0xff800000u;                   // -inf
+                        if (!(col <= hi_col && (col >= lo_col || col < keep_col))) sv[i] = 0xff800000u;                   // -inf
                     }
                 }
                 float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};     // four chains instead of one
@@ -700,16 +695,11 @@ attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
     const int ctx = kv_len - q_len;
     const int rows_here = min(NT * BM, nrows - row0);
     const int tok_lo = row0 / G, tok_hi = (row0 + rows_here - 1) / G;
-    int key_hi = ctx + tok_hi + 1;                               // exclusive
-    int key_lo = first_visible_key(ctx + tok_lo, p.window, p.chunk);
+    const KeySpan span = visible_span(ctx + tok_lo, ctx + tok_hi + 1, p.window, p.chunk, p.keep, BNK);
     const int split = blockIdx.y;
-    if (p.num_splits > 1) {
-        const int piece = piece_len(kv_len, p.num_splits, p.split_len, BN);
-        key_lo = max(key_lo, split * piece);
-        key_hi = min(key_hi, (split + 1) * piece);
-    }
-    const int t_begin = key_lo / BNK, t_end = (key_hi + BNK - 1) / BNK;
-    const int nsteps = t_end - t_begin;
+    int v_lo, v_hi;                                              // this CTA's piece, as indices into the span
+    span_piece(span, kv_len, p.window > 0 || p.chunk > 0, split, p.num_splits, p.split_len, BN, v_lo, v_hi);
+    const int nsteps = v_lo < v_hi ? (v_hi - v_lo + BNK - 1) / BNK : 0;
     if (nsteps <= 0) {
         // (only with splits) no key of this split is visible: an empty partial result, nothing allocated.  The scratch
         // memory may still be read by the merge kernel of the launch before this one: wait for it first.
@@ -788,8 +778,8 @@ attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
 #pragma unroll
                 for (int c = 0; c < BNK / 32; ++c) tmem_ld32(s_addr + c * 32, reinterpret_cast<uint32_t(&)[32]>(sv[c * 32]));
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-                const int key0 = (t_begin + j) * BNK;
-                const int hi_col = valid ? pos - key0 : -1, lo_col = lo - key0;
+                const int key0 = span.key(v_lo + j * BNK);
+                const int hi_col = valid ? pos - key0 : -1, lo_col = lo - key0, keep_col = p.keep - key0;
                 const bool tile_full = __all_sync(0xffffffffu, valid && hi_col >= BNK - 1 && lo_col <= 0);
                 if (p.cap_in != 0.f) {
 #pragma unroll
@@ -798,7 +788,7 @@ attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
                 if (!tile_full) {
 #pragma unroll
                     for (int i = 0; i < BNK; ++i)
-                        if (!(i <= hi_col && i >= lo_col)) sv[i] = 0xff800000u;                   // -inf
+                        if (!(i <= hi_col && (i >= lo_col || i < keep_col))) sv[i] = 0xff800000u;                   // -inf
                 }
                 float mx8[8];
 #pragma unroll
@@ -952,7 +942,7 @@ attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
             auto box_row = [&](int j) -> int {                  // first row of this lane's box of tile j in the page matrix
                 int y = 0;
                 if (lane < nboxes && j < nsteps) {
-                    const int key = (t_begin + j) * BNK + lane * box_rows;
+                    const int key = span.key(v_lo + j * BNK) + lane * box_rows;
                     const int pg = key / ps;
                     const int page = pg < p.table_width ? table[pg] : 0;
                     y = (page * p.Hkv + kvh) * ps + (key - pg * ps);
@@ -1195,7 +1185,7 @@ extern "C" int ttie_attn_tc_supported(int D, int page_size) {
 extern "C" int ttie_paged_attention_tc_weights(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
                                                int num_pages, const int* block_table, int table_width, int page_size, const int* qsl,
                                                const int* seq_lens, void* out, int T, int num_seqs, int Hq, int Hkv, int D,
-                                               int max_q_len, float scale, float softcap, int window, int chunk, int num_splits, int split_len,
+                                               int max_q_len, float scale, float softcap, int window, int chunk, int keep, int num_splits, int split_len,
                                                float* scratch, int two_tiles, int weights, const float* head_bias, void* stream);
 
 extern "C" int ttie_paged_attention_tc(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
@@ -1204,14 +1194,14 @@ extern "C" int ttie_paged_attention_tc(const void* q, long long q_stride, const 
                                        int max_q_len, float scale, float softcap, int window, int chunk, int num_splits, int split_len, float* scratch,
                                        int two_tiles, void* stream) {
     return ttie_paged_attention_tc_weights(q, q_stride, k_pages, v_pages, num_pages, block_table, table_width, page_size, qsl, seq_lens, out, T,
-                                           num_seqs, Hq, Hkv, D, max_q_len, scale, softcap, window, chunk, num_splits, split_len, scratch,
+                                           num_seqs, Hq, Hkv, D, max_q_len, scale, softcap, window, chunk, 0, num_splits, split_len, scratch,
                                            two_tiles, 0, nullptr, stream);
 }
 
 extern "C" int ttie_paged_attention_tc_weights(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
                                                int num_pages, const int* block_table, int table_width, int page_size, const int* qsl,
                                                const int* seq_lens, void* out, int T, int num_seqs, int Hq, int Hkv, int D,
-                                               int max_q_len, float scale, float softcap, int window, int chunk, int num_splits, int split_len,
+                                               int max_q_len, float scale, float softcap, int window, int chunk, int keep, int num_splits, int split_len,
                                                float* scratch, int two_tiles, int weights, const float* head_bias, void* stream) {
     if (T <= 0 || num_seqs <= 0) return 0;
     if (weights != 0 && weights != 1) TTIE_FAIL("attention_tc: unknown kind of weights %d", weights);
@@ -1234,6 +1224,7 @@ extern "C" int ttie_paged_attention_tc_weights(const void* q, long long q_stride
     p.q = (const __nv_bfloat16*)q; p.q_stride = q_stride; p.block_table = block_table; p.table_width = table_width;
     p.page_size = page_size; p.qsl = qsl; p.seq_lens = seq_lens; p.out = (__nv_bfloat16*)out;
     p.num_seqs = num_seqs; p.Hq = Hq; p.Hkv = Hkv; p.scale_log2 = scale * 1.4426950408889634f; p.window = window; p.chunk = chunk;
+    p.keep = window > 0 ? keep : 0;
     p.cap_in = softcap > 0.f ? scale / softcap : 0.f; p.cap_out = softcap > 0.f ? softcap / scale : 0.f;
     p.row_tiles = ceil_div(max_q_len * (Hq / Hkv), two_tiles && D <= 128 ? 2 * BM : BM);
     p.num_splits = num_splits; p.split_len = split_len;

@@ -45,6 +45,33 @@ __device__ __forceinline__ int first_visible_key(int pos, int window, int chunk)
     return window > 0 ? max(0, pos - window + 1) : 0;
 }
 
+// The keys that a tile of query rows walks, as one run of indices 0 .. total-1: with a window whose sequence keeps its first
+// `keep` tokens visible the keys are two ranges, [0, keep) and [first visible key of the lowest row, k_hi), and index v stands
+// for key  v < kept ? v : v - kept + first.  Both ranges start on multiples of `granule` (the kernel's key tile), so a tile
+// never straddles them; the mask cuts what the rounding adds.  Without kept tokens kept = 0; where the ranges meet they are one.
+struct KeySpan {
+    int first, kept, total;
+    __device__ __forceinline__ int key(int v) const { return v < kept ? v : v - kept + first; }
+};
+__device__ __forceinline__ KeySpan visible_span(int pos_lo, int k_hi, int window, int chunk, int keep, int granule) {
+    KeySpan s;
+    s.first = first_visible_key(pos_lo, window, chunk) / granule * granule;
+    s.kept = keep > 0 ? min((keep + granule - 1) / granule * granule, s.first) : 0;
+    s.total = s.kept + max(0, k_hi - s.first);
+    return s;
+}
+// The indices [lo, hi) of piece `split` of a span that was planned as num_splits pieces of split_len.  Without a window or a
+// chunk the share is that of the request's whole length, the same for each of its row tiles.
+__device__ __forceinline__ void span_piece(const KeySpan& s, int kv_len, bool bounded, int split, int num_splits, int split_len, int granule,
+                                           int& lo, int& hi) {
+    lo = 0; hi = s.total;
+    if (num_splits > 1) {
+        const int piece = piece_len(bounded ? s.total : kv_len, num_splits, split_len, granule);
+        lo = split * piece;
+        hi = min(hi, lo + piece);
+    }
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

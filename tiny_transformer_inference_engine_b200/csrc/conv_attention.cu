@@ -39,6 +39,7 @@ struct QkvArgs {
                                                                     // all heads at once; norm_w is then [Hq*D + Hkv*D], a weight per channel); null: a norm per head
     int v_from_k;                                                   // the values are the key heads before norm and rotation
     float qt_coef; int qt_every;                                    // query temperature; every 0: none
+    const void* v_first; long long ld_first; float v_mix;           // values become (1 - v_mix) * v + v_mix * v_first; null: as they are
     void* q_out; void* k_pages; void* v_pages;
     const int* block_table; int table_width, page_size, num_pages, write_kv;
 };
@@ -136,8 +137,12 @@ __global__ void __launch_bounds__(128) qkv_conv_rope_store_kernel(const QkvArgs 
             kp[i] = from_f32<T>(i < a.D ? rotated(row, i, a.rot, a.style, cs) : 0.f);
     } else {
         T* vp = reinterpret_cast<T*>(a.v_pages) + dst;
-        for (int i = threadIdx.x; i < a.Dp; i += blockDim.x)
-            vp[i] = from_f32<T>(i < a.Dv ? row[i] : 0.f);
+        const T* vf = a.v_first ? reinterpret_cast<const T*>(a.v_first) + (size_t)t * a.ld_first + (size_t)h * a.Dv : nullptr;
+        for (int i = threadIdx.x; i < a.Dp; i += blockDim.x) {
+            float v = i < a.Dv ? row[i] : 0.f;
+            if (vf && i < a.Dv) v = (1.0f - a.v_mix) * v + a.v_mix * to_f32(vf[i]);
+            vp[i] = from_f32<T>(v);
+        }
     }
 }
 
@@ -248,6 +253,11 @@ __global__ void __launch_bounds__(256) qkv_conv_rope_store_vec8_kernel(const Qkv
                 out[i] = x * c.x - y * c.y; out[i + 1] = x * c.y + y * c.x;
             }
         }
+    }
+    if (kind == 2 && inside && a.v_first) {
+        const __nv_bfloat16* vf = reinterpret_cast<const __nv_bfloat16*>(a.v_first) + (size_t)t * a.ld_first + (size_t)h * a.Dv + i0;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) out[i] = (1.0f - a.v_mix) * out[i] + a.v_mix * __bfloat162float(vf[i]);
     }
     const int pos = a.positions[t];
     if (kind == 0 && a.qt_every > 0) {
@@ -423,7 +433,7 @@ extern "C" int ttie_qkv_conv_rope_store(const void* proj, long long ld, int T, i
                                         const float* conv_w, const float* tail, int tail_rows, const int* positions,
                                         const int* token_seq, const int* qsl, const int* slot_ids, const void* cs, int rot, int style,
                                         const float* norm_w, float norm_eps, const float* row_inv, int v_from_k, float qt_coef, int qt_every,
-                                        void* q_out, void* k_pages, void* v_pages, const int* block_table, int table_width,
+                                        const void* v_first, long long ld_first, float v_mix, void* q_out, void* k_pages, void* v_pages, const int* block_table, int table_width,
                                         int page_size, int num_pages, int write_kv, int dtype, void* stream) {
     if (T <= 0) return 0;
     if (v_from_k && Dv != D) TTIE_FAIL("qkv_conv_rope_store: values that are the keys have the keys' size, not %d against %d", Dv, D);
@@ -437,7 +447,7 @@ extern "C" int ttie_qkv_conv_rope_store(const void* proj, long long ld, int T, i
     a.proj = proj; a.ld = ld; a.Hq = Hq; a.Hkv = Hkv; a.D = D; a.Dv = Dv; a.Dp = Dp; a.taps = taps; a.conv_w = conv_w; a.tail = tail;
     a.tail_rows = tail_rows; a.positions = positions; a.token_seq = token_seq; a.qsl = qsl; a.slot_ids = slot_ids;
     a.cs = (const float2*)cs; a.rot = rot; a.style = style; a.norm_w = norm_w; a.norm_eps = norm_eps; a.row_inv = row_inv; a.v_from_k = v_from_k;
-    a.qt_coef = qt_coef; a.qt_every = qt_every; a.q_out = q_out; a.k_pages = k_pages; a.v_pages = v_pages;
+    a.qt_coef = qt_coef; a.qt_every = qt_every; a.v_first = v_first; a.ld_first = ld_first; a.v_mix = v_mix; a.q_out = q_out; a.k_pages = k_pages; a.v_pages = v_pages;
     a.block_table = block_table; a.table_width = table_width; a.page_size = page_size; a.num_pages = num_pages; a.write_kv = write_kv;
     const size_t smem = (size_t)(D > Dv ? D : Dv) * sizeof(float);
     if (T > 2147483647 / 1 || Hq + 2 * Hkv > 65535) TTIE_FAIL("qkv_conv_rope_store: %d heads exceed the grid", Hq + 2 * Hkv);

@@ -786,6 +786,34 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const T* __re
     }
 }
 
+// the same for long rows (a norm over all heads at once): one CTA per row, the row in registers
+template <typename T, int PER>
+__global__ void __launch_bounds__(256) row_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ gate, long long ld_g, const float* __restrict__ w,
+                                                            int n, float eps, int act, T* __restrict__ out) {
+    __shared__ float scratch[32];
+    TTIE_PDL_ENTRY();
+    const float* src = o + (size_t)blockIdx.x * n;
+    const T* gp = gate + (size_t)blockIdx.x * ld_g;
+    float v[PER], g[PER];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int j = threadIdx.x + k * blockDim.x;
+        v[k] = j < n ? src[j] : 0.f;
+        g[k] = j < n ? to_f32(gp[j]) : 0.f;
+        ss = fmaf(v[k], v[k], ss);
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)n + eps);
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int j = threadIdx.x + k * blockDim.x;
+        if (j >= n) continue;
+        const float sg = 1.0f / (1.0f + expf(-g[k]));
+        out[(size_t)blockIdx.x * n + j] = from_f32<T>(v[k] * inv * (w ? w[j] : 1.0f) * (act == 0 ? g[k] * sg : sg));
+    }
+}
+
 // Key channels per thread for heads of D key channels: the fewest (the most threads per state) whose slices still fit a warp.
 int keys_per_thread(int D) { return D <= 128 ? 4 : D <= 256 ? 8 : 16; }
 
@@ -974,6 +1002,16 @@ extern "C" int ttie_head_norm_gate(const float* o, const void* gate, long long l
                                    int act, void* out, int dtype, void* stream) {
     if (T <= 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
+    if (H == 1 && Dv > 256 && Dv <= 8192) {
+        if (dtype != kF32 && dtype != kBF16) TTIE_FAIL("head_norm_gate: unknown dtype %d", dtype);
+#define RNG(TT, PER) TTIE_LAUNCH((row_norm_gate_kernel<TT, PER>), T, 256, 0, s, o, (const TT*)gate, ld_g, w, Dv, eps, act, (TT*)out)
+        if (Dv <= 1024) { if (dtype == kF32) RNG(float, 4); else RNG(__nv_bfloat16, 4); }
+        else if (Dv <= 4096) { if (dtype == kF32) RNG(float, 16); else RNG(__nv_bfloat16, 16); }
+        else { if (dtype == kF32) RNG(float, 32); else RNG(__nv_bfloat16, 32); }
+#undef RNG
+        TTIE_CHECK_LAUNCH("head_norm_gate");
+        return 0;
+    }
     const long long units = (long long)T * H;
     const int grid = (int)((units + 7) / 8);
     if (dtype == kF32) TTIE_LAUNCH(head_norm_gate_kernel<float>, grid, 256, 0, s, o, (const float*)gate, ld_g, w, T, H, Dv, eps, act, (float*)out);

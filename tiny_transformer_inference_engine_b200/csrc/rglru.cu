@@ -1,8 +1,9 @@
 // The recurrent block with a real-gated linear recurrent unit (RG-LRU), for any split of a sequence into steps.
 // Per request the state row holds [taps, width] 32-bit values: row 0 is the recurrent state S, rows 1 .. taps-1 the last
 // taps-1 inputs of the short convolution (oldest first).
-//   causal_conv:  u[t, c] = sum_k w[k, c] * in[t - (taps-1) + k, c] + b[c]   (weights tap-major; inputs before the step come from the state row,
-//                 zeros before the sequence's start because a fresh row is zero); one thread per (token, channel)
+//   causal_conv:  u[t, c] = act(sum_k w[k, c] * in[t - (taps-1) + k, c] + b[c])   (weights tap-major; inputs before the step come from the
+//                 state row, zeros before the sequence's start because a fresh row is zero; act: none here, or silu); one thread
+//                 per (token, channel).  Where the taps-1 earlier inputs lie in a state row is the caller's: row stride and offset
 //   rglru_scan:   r = sigmoid(pre_r + br), i = sigmoid(pre_i + bi), log a = -c * r * softplus(lam), a = exp(log a),
 //                 S <- a * S + sqrt(1 - a^2) * i * u,  out = S * gelu_tanh(y_pre); all 32-bit; it also moves the convolution's
 //                 inputs of this step into the state row.  Two forms: one thread per (request, channel) walking the tokens
@@ -24,7 +25,7 @@ __device__ __forceinline__ int slot_row(int slot, int num_rows) { return slot < 
 template <typename T, typename W>
 __global__ void causal_conv_kernel(const T* __restrict__ in, long long ld, int col0, int T_, int width, int taps,
                                    const W* __restrict__ cw, const W* __restrict__ cb, const float* __restrict__ state,
-                                   int state_rows, const int* __restrict__ token_seq, const int* __restrict__ qsl,
+                                   int state_rows, long long row_stride, int tail_off, int silu, const int* __restrict__ token_seq, const int* __restrict__ qsl,
                                    const int* __restrict__ slot_ids, float* __restrict__ u32, T* __restrict__ u_c) {
     TTIE_PDL_ENTRY();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;             // grid: (channels, tokens)
@@ -33,14 +34,15 @@ __global__ void causal_conv_kernel(const T* __restrict__ in, long long ld, int c
         const size_t e = (size_t)t * width + c;
         const int s = token_seq[t];
         const int j = t - qsl[s];                                   // index within the request's tokens of this step
-        const float* tail = state + ((size_t)slot_row(slot_ids[s], state_rows) * taps + 1) * width;
+        const float* tail = state + (size_t)slot_row(slot_ids[s], state_rows) * row_stride + tail_off;
         float acc = cb ? to_f32(cb[c]) : 0.f;
         for (int k = 0; k < taps; ++k) {
             const int src = j - (taps - 1) + k;
             const float v = src >= 0 ? to_f32(in[(size_t)(t - j + src) * ld + col0 + c]) : tail[(size_t)(taps - 1 + src) * width + c];
             acc = fmaf(to_f32(cw[(size_t)k * width + c]), v, acc);
         }
-        u32[e] = acc;
+        if (silu) acc *= sigmoidf_(acc);
+        if (u32) u32[e] = acc;
         if (u_c) u_c[e] = from_f32<T>(acc);
     }
 }
@@ -61,7 +63,7 @@ template <typename W>
 __global__ void __launch_bounds__(128)
 causal_conv_vec8_kernel(const __nv_bfloat16* __restrict__ in, long long ld, int col0, int T_, int width, int taps,
                         const W* __restrict__ cw, const W* __restrict__ cb, const float* __restrict__ state, int state_rows,
-                        const int* __restrict__ token_seq, const int* __restrict__ qsl, const int* __restrict__ slot_ids,
+                        long long row_stride, int tail_off, int silu, const int* __restrict__ token_seq, const int* __restrict__ qsl, const int* __restrict__ slot_ids,
                         float* __restrict__ u32, __nv_bfloat16* __restrict__ u_c) {
     TTIE_PDL_ENTRY();
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
@@ -69,7 +71,7 @@ causal_conv_vec8_kernel(const __nv_bfloat16* __restrict__ in, long long ld, int 
     for (int t = blockIdx.y; t < T_; t += gridDim.y) {
         const int s = token_seq[t];
         const int j = t - qsl[s];
-        const float* tail = state + ((size_t)slot_row(slot_ids[s], state_rows) * taps + 1) * width;
+        const float* tail = state + (size_t)slot_row(slot_ids[s], state_rows) * row_stride + tail_off;
         float acc[8];
         if (cb) load8(cb + c, acc);
         else {
@@ -94,9 +96,15 @@ causal_conv_vec8_kernel(const __nv_bfloat16* __restrict__ in, long long ld, int 
 #pragma unroll
             for (int i = 0; i < 8; ++i) acc[i] = fmaf(w[i], v[i], acc[i]);
         }
-        float* o = u32 + (size_t)t * width + c;
-        *reinterpret_cast<float4*>(o) = make_float4(acc[0], acc[1], acc[2], acc[3]);
-        *reinterpret_cast<float4*>(o + 4) = make_float4(acc[4], acc[5], acc[6], acc[7]);
+        if (silu) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) acc[i] *= sigmoidf_(acc[i]);
+        }
+        if (u32) {
+            float* o = u32 + (size_t)t * width + c;
+            *reinterpret_cast<float4*>(o) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+            *reinterpret_cast<float4*>(o + 4) = make_float4(acc[4], acc[5], acc[6], acc[7]);
+        }
         if (u_c) {
             uint4 p;
             __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&p);
@@ -345,23 +353,25 @@ inline int grid_for(size_t total) { return (int)((total + 255) / 256 < 8192 ? (t
 }  // namespace
 
 extern "C" int ttie_causal_conv(const void* in, long long ld, int col0, int T, int width, int taps, const void* cw, const void* cb,
-                                int w_dtype, const float* state, int state_rows, const int* token_seq, const int* qsl,
+                                int w_dtype, const float* state, int state_rows, long long row_stride, int tail_off, int silu, const int* token_seq, const int* qsl,
                                 const int* slot_ids, float* u32, void* u_c, int dtype, void* stream) {
     if (T <= 0) return 0;
     if (taps < 1) TTIE_FAIL("causal_conv: %d taps", taps);
+    if (taps > 1 && !state) TTIE_FAIL("causal_conv: %d taps need state rows", taps);
+    if (!u32 && !u_c) TTIE_FAIL("causal_conv: no output");
     cudaStream_t s = (cudaStream_t)stream;
-    if (dtype == kBF16 && width % 8 == 0 && ld % 8 == 0 && col0 % 8 == 0 && ((((uintptr_t)in) | ((uintptr_t)state) | ((uintptr_t)u32) | ((uintptr_t)u_c) | ((uintptr_t)cw) | ((uintptr_t)cb)) & 15) == 0) {
+    if (dtype == kBF16 && width % 8 == 0 && ld % 8 == 0 && col0 % 8 == 0 && row_stride % 4 == 0 && tail_off % 4 == 0 && ((((uintptr_t)in) | ((uintptr_t)state) | ((uintptr_t)u32) | ((uintptr_t)u_c) | ((uintptr_t)cw) | ((uintptr_t)cb)) & 15) == 0) {
         const dim3 g8(ceil_div(width / 8, 128), T < 65535 ? T : 65535);
         if (w_dtype == kF32) TTIE_LAUNCH(causal_conv_vec8_kernel<float>, g8, 128, 0, s, (const __nv_bfloat16*)in, ld, col0, T, width, taps, (const float*)cw,
-                                         (const float*)cb, state, state_rows, token_seq, qsl, slot_ids, u32, (__nv_bfloat16*)u_c);
+                                         (const float*)cb, state, state_rows, row_stride, tail_off, silu, token_seq, qsl, slot_ids, u32, (__nv_bfloat16*)u_c);
         else TTIE_LAUNCH(causal_conv_vec8_kernel<__nv_bfloat16>, g8, 128, 0, s, (const __nv_bfloat16*)in, ld, col0, T, width, taps, (const __nv_bfloat16*)cw,
-                         (const __nv_bfloat16*)cb, state, state_rows, token_seq, qsl, slot_ids, u32, (__nv_bfloat16*)u_c);
+                         (const __nv_bfloat16*)cb, state, state_rows, row_stride, tail_off, silu, token_seq, qsl, slot_ids, u32, (__nv_bfloat16*)u_c);
         TTIE_CHECK_LAUNCH("causal_conv");
         return 0;
     }
     const dim3 grid(ceil_div(width, 256), T < 65535 ? T : 65535);
 #define CC(TT, WW) TTIE_LAUNCH((causal_conv_kernel<TT, WW>), grid, 256, 0, s, (const TT*)in, ld, col0, T, width, taps, (const WW*)cw, \
-                               (const WW*)cb, state, state_rows, token_seq, qsl, slot_ids, u32, (TT*)u_c)
+                               (const WW*)cb, state, state_rows, row_stride, tail_off, silu, token_seq, qsl, slot_ids, u32, (TT*)u_c)
     if (dtype == kF32) { if (w_dtype != kF32) TTIE_FAIL("causal_conv: a 32-bit run needs 32-bit weights"); CC(float, float); }
     else if (w_dtype == kF32) CC(__nv_bfloat16, float);
     else CC(__nv_bfloat16, __nv_bfloat16);

@@ -75,9 +75,8 @@ class BatchPacker:
                 table = g.tables.get(en.rid)
                 if table is None:
                     raise KeyError(f"request {en.rid!r} is not admitted")
-                first = g.first_needed_page(en.start)
                 last = -(-(en.start + n) // g.page_size)
-                span = table[first:last]
+                span = [table[i] for i in g.needed_pages(en.start, min(last, len(table)))] if g.reach is not None else table[:last]
                 if len(table) < last or (span and (min(span) <= 0 or max(span) >= g.num_pages)):
                     raise ValueError(f"request {en.rid!r}: block table of group {gi} does not cover "
                                      f"positions {en.start}..{en.start + n - 1}")

@@ -102,7 +102,8 @@ class Model:
             self.blocks[entry.layer].forward(stream, ctx, cache_views[e])
             if self.after_entry is not None:                     # (a debugging aid: sees the stream after every run entry)
                 self.after_entry(e, stream)
-        x = self.final_norm.norm_rows(stream.resid, stream.delta, ctx.logit_rows, ctx.num_logit_rows)
+        pending = {} if stream.delta_norm is None else {"delta_norm": stream.delta_norm}
+        x = self.final_norm.norm_rows(stream.resid, stream.delta, ctx.logit_rows, ctx.num_logit_rows, **pending)
         if ctx.num_logit_rows == 0:
             return torch.empty((0, self.spec.vocab_size), dtype=torch.float32, device=ctx.device)
         return self.head.forward(x)

@@ -52,16 +52,16 @@ _SIGNATURES = {
                                       _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_int, _c_int, _c_int,
                                       _c_void, _c_int, _c_void],
     "ttie_paged_attention_weights": [_c_void, _c_ll, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_void, _c_void,
-                                     _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_int, _c_int, _c_int,
+                                     _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_int, _c_int, _c_int, _c_int,
                                      _c_void, _c_int, _c_int, _c_void, _c_void],
     "ttie_paged_attention_mma_weights": [_c_void, _c_ll, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_void, _c_void,
-                                         _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_int, _c_int, _c_int,
+                                         _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_int, _c_int, _c_int, _c_int,
                                          _c_void, _c_int, _c_int, _c_void, _c_void],
     "ttie_paged_attention_tc": [_c_void, _c_ll, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_void, _c_void, _c_void,
                                 _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int,
                                 _c_void],
     "ttie_paged_attention_tc_weights": [_c_void, _c_ll, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_void, _c_void, _c_void,
-                                        _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int,
+                                        _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int,
                                         _c_int, _c_void, _c_void],
     "ttie_gemm_tc": [_c_void, _c_ll, _c_void, _c_ll, _c_void, _c_void, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void],
     "ttie_gemm_tc_pair": [_c_void, _c_ll, _c_void, _c_ll, _c_void, _c_void, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void],
@@ -74,8 +74,23 @@ _SIGNATURES = {
     "ttie_gate_heads": [_c_void, _c_void, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int, _c_void],
     "ttie_rmsnorm_cols": [_c_void, _c_ll, _c_int, _c_int, _c_int, _c_void, _c_int, _c_float, _c_void, _c_int, _c_void],
     "ttie_gemm_f32_batched": [_c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_ll, _c_ll, _c_ll, _c_ll, _c_ll, _c_ll, _c_void],
-    "ttie_causal_conv": [_c_void, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_int, _c_void, _c_int, _c_void, _c_void,
-                         _c_void, _c_void, _c_void, _c_int, _c_void],
+    "ttie_causal_conv": [_c_void, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_int, _c_void, _c_int, _c_ll, _c_int, _c_int,
+                         _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_void],
+    "ttie_selective_scan": [_c_void, _c_ll, _c_void, _c_ll, _c_void, _c_void, _c_void, _c_void, _c_ll, _c_int, _c_int, _c_void, _c_ll,
+                            _c_void, _c_int, _c_void, _c_ll, _c_void, _c_int, _c_int, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_int,
+                            _c_void, _c_int, _c_void],
+    "ttie_selective_state_pad": [_c_int],
+    "ttie_sandwich_norm": [_c_void, _c_void, _c_void, _c_int, _c_ll, _c_void, _c_void, _c_float, _c_void, _c_float, _c_void, _c_int, _c_int,
+                           _c_int, _c_void],
+    "ttie_joint_store_supported": [_c_int, _c_int, _c_int],
+    "ttie_joint_qkv_store": [_c_void, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_float, _c_void, _c_int, _c_int,
+                             _c_void, _c_ll, _c_float, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_void,
+                             _c_int, _c_void],
+    "ttie_joint_values": [_c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void],
+    "ttie_attn_joint_tile_rows": [_c_int, _c_int],
+    "ttie_paged_attention_joint": [_c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int,
+                                   _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int, _c_void],
+    "ttie_activation_rows": [_c_void, _c_ll, _c_void, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_void],
     "ttie_rglru_scan": [_c_void, _c_void, _c_void, _c_void, _c_int, _c_void, _c_void, _c_ll, _c_int, _c_void, _c_ll, _c_int, _c_void,
                         _c_int, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void, _c_int, _c_void,
                         _c_int, _c_void],
@@ -94,7 +109,7 @@ _SIGNATURES = {
     "ttie_moe_combine": [_c_void, _c_int, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_void, _c_int, _c_void, _c_int, _c_void, _c_ll, _c_void],
     "ttie_qkv_conv_rope_store": [_c_void, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_int, _c_void,
                                  _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_float, _c_void, _c_int, _c_float, _c_int,
-                                 _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void],
+                                 _c_void, _c_ll, _c_float, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void],
     "ttie_proj_row_rms": [_c_void, _c_ll, _c_int, _c_int, _c_int, _c_float, _c_void, _c_int, _c_void],
     "ttie_stream_conv": [_c_void, _c_int, _c_int, _c_int, _c_void, _c_void, _c_int, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void],
     "ttie_conv_tail_update": [_c_void, _c_ll, _c_int, _c_int, _c_void, _c_int, _c_void, _c_void, _c_int, _c_int, _c_void],
@@ -112,7 +127,7 @@ _SIGNATURES = {
     "ttie_retention_scan": [_c_void, _c_void, _c_ll, _c_void, _c_ll, _c_void, _c_void, _c_int, _c_void, _c_void, _c_int, _c_void, _c_int,
                             _c_int, _c_int, _c_int, _c_void, _c_int, _c_void],
     "ttie_head_norm_gate": [_c_void, _c_void, _c_ll, _c_void, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void, _c_int, _c_void],
-    "ttie_activation": [_c_void, _c_void, _c_ll, _c_int, _c_float, _c_int, _c_int, _c_void],
+    "ttie_activation": [_c_void, _c_void, _c_ll, _c_int, _c_float, _c_float, _c_int, _c_int, _c_void],
     "ttie_matrix_state_pad": [_c_int],
     "ttie_sample": [_c_void, _c_int, _c_int, _c_void, _c_void, _c_void, _c_void, _c_void],
     "ttie_sample_tuned": [_c_void, _c_int, _c_int, _c_void, _c_void, _c_void, _c_void, _c_int, _c_void],
@@ -276,6 +291,17 @@ class CudaOps:
         self._check(self.lib.ttie_add_rmsnorm(_ptr(resid), dp, pp, S, stride, _ptr(rows), _ptr(weight), self._dt(weight),
                                               _ptr(out), num_rows, d, float(eps), self._dt(out), self._stream(out)),
                     "rmsnorm_rows")
+        self.launches += 1
+
+    def sandwich_norm(self, resid, delta, delta_weight, delta_eps, weight, eps, out, rows=None, num_rows=None):
+        """resid <- resid + rms_norm(delta) * delta_weight over the 32-bit stream [R, d], and out = rms_norm(resid) * weight in the
+        compute dtype, in one pass.  ``delta``: [R, d] or float32 partial sums [S, R, d]; weights float32 [d].  With ``rows`` the
+        rows are gathered into ``out`` [num_rows, d] and the stream is left alone."""
+        d = resid.shape[1]
+        dp, pp, S, stride = self._delta_args(delta)
+        self._check(self.lib.ttie_sandwich_norm(_ptr(resid), dp, pp, S, stride, _ptr(rows), _ptr(delta_weight), float(delta_eps),
+                                                _ptr(weight), float(eps), _ptr(out), resid.shape[0] if rows is None else int(num_rows), d,
+                                                self._dt(out), self._stream(out)), "sandwich_norm")
         self.launches += 1
 
     # ---- matrix products
@@ -819,9 +845,9 @@ class CudaOps:
 
     def paged_attention(self, qkv, num_heads, num_kv_heads, head_dim, k_pages, v_pages, block_table, page_size,
                         query_start_loc, seq_lens, num_seqs, max_q_len, max_kv_len, scale, window, out,
-                        plan=None, softcap=0.0, chunk=0, weights="softmax", head_bias=None):
+                        plan=None, softcap=0.0, chunk=0, weights="softmax", head_bias=None, keep_first=0):
         """Causal attention of the step's query rows over the paged keys and values.  ``window`` > 0: a row at position p
-        sees keys p - window + 1 .. p.  ``chunk`` > 0 (instead of a window): a row at position p sees the keys of its own
+        sees keys p - window + 1 .. p, and with ``keep_first`` > 0 also the sequence's first ``keep_first`` keys.  ``chunk`` > 0 (instead of a window): a row at position p sees the keys of its own
         chunk of ``chunk`` positions up to p, chunks counted from position 0 of the sequence.  ``softcap`` > 0: a score s
         (scale applied) becomes softcap * tanh(s / softcap) before mask and softmax.  ``weights`` "sigmoid": a visible key
         weighs sigmoid(score + head_bias[head]) (``head_bias`` float32 [num_heads] or None) and nothing is normalised over the
@@ -835,7 +861,8 @@ class CudaOps:
         if max_kv_len > block_table.shape[1] * page_size:
             raise KernelError(f"paged_attention: a block table of {block_table.shape[1]} pages of {page_size} keys cannot cover {max_kv_len} keys")
         kernel, num_splits, split_len = plan if plan is not None else self.attention_plan(
-            qkv.dtype, num_seqs, num_heads, num_kv_heads, head_dim, max_q_len, max_kv_len, page_size, sig)
+            qkv.dtype, num_seqs, num_heads, num_kv_heads, head_dim, max_q_len, self.visible_keys(max_q_len, max_kv_len, window, chunk, keep_first),
+            page_size, sig)
         if sig and kernel not in ("mma", "simt", "tc", "tcpp"):
             raise KernelError(f"paged_attention: sigmoid weights have no {kernel!r} kernel")
         if kernel in ("tc", "tcpp"):
@@ -845,7 +872,7 @@ class CudaOps:
             self._check(self.lib.ttie_paged_attention_tc_weights(
                 _ptr(qkv), qkv.stride(0), _ptr(k_pages), _ptr(v_pages), k_pages.shape[0], _ptr(block_table),
                 block_table.shape[1], page_size, _ptr(query_start_loc), _ptr(seq_lens), _ptr(out), T, num_seqs, num_heads,
-                num_kv_heads, head_dim, max_q_len, float(scale), float(softcap or 0.0), int(window), int(chunk), num_splits, split_len, _ptr(scratch),
+                num_kv_heads, head_dim, max_q_len, float(scale), float(softcap or 0.0), int(window), int(chunk), int(keep_first), num_splits, split_len, _ptr(scratch),
                 1 if kernel == "tcpp" else 0, 1 if sig else 0, _ptr(head_bias), self._stream(qkv)), "paged_attention_tc")
             self.launches += 2 if num_splits > 1 else 1
             return
@@ -857,7 +884,7 @@ class CudaOps:
             self._check(self.lib.ttie_paged_attention_mma_weights(
                 _ptr(qkv), qkv.stride(0), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1],
                 page_size, _ptr(query_start_loc), _ptr(seq_lens), _ptr(out), T, num_seqs, num_heads, num_kv_heads,
-                head_dim, max_q_len, float(scale), float(softcap or 0.0), int(window), int(chunk), num_splits, split_len, _ptr(scratch),
+                head_dim, max_q_len, float(scale), float(softcap or 0.0), int(window), int(chunk), int(keep_first), num_splits, split_len, _ptr(scratch),
                 form, 1 if sig else 0, _ptr(head_bias), self._stream(qkv)), "paged_attention_mma")
             self.launches += 2 if (num_splits > 1 and not form) else 1
             return
@@ -865,8 +892,97 @@ class CudaOps:
             self._check(self.lib.ttie_paged_attention_weights(
                 _ptr(qkv), qkv.stride(0), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1],
                 page_size, _ptr(query_start_loc), _ptr(seq_lens), _ptr(out), T, num_seqs, num_heads, num_kv_heads,
-                head_dim, max_q_len, float(scale), float(softcap or 0.0), int(window), int(chunk), num_splits, split_len, _ptr(scratch),
+                head_dim, max_q_len, float(scale), float(softcap or 0.0), int(window), int(chunk), int(keep_first), num_splits, split_len, _ptr(scratch),
                 self._dt(qkv), 1 if sig else 0, _ptr(head_bias), self._stream(qkv)), "paged_attention")
+        self.launches += 2 if num_splits > 1 else 1
+
+    @staticmethod
+    def visible_keys(max_q_len, max_kv_len, window, chunk, keep_first):
+        """The most keys that a request's rows of a step walk (with the kernels' rounding to tiles of 128 keys): what the key
+        range is planned for.  A window's or a chunk's rows start at their lowest row's first key, whatever the context."""
+        reach = window or chunk
+        if not reach:
+            return max_kv_len
+        kept = -(-keep_first // 128) * 128 if window and keep_first else 0
+        return min(max_kv_len, kept + reach + max_q_len + 127)
+
+    # ---- attention whose scores are mixed over the heads: joint rows of all kv heads
+    def joint_width(self, dtype, kv_heads, head_dim, v_dim) -> int:
+        """Values of a joint key / value row: room for all kv heads' keys and for their values, padded to what the attention
+        kernels take (bfloat16: multiples of 16 up to 128, then 256, else multiples of 8; float32: multiples of 4)."""
+        need = kv_heads * max(head_dim, v_dim)
+        if dtype == torch.float32:
+            return -(-need // 4) * 4
+        if need <= 128:
+            return -(-need // 16) * 16
+        return 256 if need <= 256 else -(-need // 8) * 8
+
+    def check_joint_attention(self, dtype, num_heads, kv_heads, head_dim, v_dim, page_size):
+        """Raises unless the joint-row kernels take the sizes."""
+        self.check_dtype(dtype)
+        W = self.joint_width(dtype, kv_heads, head_dim, v_dim)
+        if not self.lib.ttie_attn_joint_tile_rows(W, v_dim) or not self.lib.ttie_joint_store_supported(num_heads, kv_heads, head_dim):
+            raise KernelError(f"mixed heads: {num_heads} heads on {kv_heads} kv heads of {head_dim} / {v_dim} values are not supported")
+        if page_size < 1:
+            raise KernelError(f"attention: page size {page_size}")
+
+    def joint_qkv_store(self, proj, num_heads, kv_heads, head_dim, v_dim, width, mix, positions, token_seq, cs_table, rot, style,
+                        k_pages, v_pages, block_table, page_size, write_kv, norm_w=None, norm_eps=0.0, v_first=None, v_mix=0.0):
+        """From a step's projected rows ``proj`` [T, >= H*D + G*D + G*Dv] (columns [q | k | v]): one norm over all of q and one over
+        all of k (``norm_w`` float32 [H*D + G*D] or None), the rotation of the first ``rot`` values of every head, and the joint
+        rows: a query row [G*D] per head that holds, for every kv head, the sum of its query heads' rows with the head's weights of
+        ``mix`` (float32 [H, H] TRANSPOSED: mix[g, h] weighs head g's scores in head h's); keys and values of all kv heads side by side
+        into the pages [pages, 1, page, width].  ``v_first`` (a view [T, G*Dv] with a row stride): values are stored as
+        (1 - v_mix) * v + v_mix * v_first.  Returns q [T, H * width]."""
+        T = proj.shape[0]
+        q = torch.empty((T, num_heads * width), dtype=proj.dtype, device=proj.device)
+        self._check(self.lib.ttie_joint_qkv_store(
+            _ptr(proj), proj.stride(0), T, num_heads, kv_heads, head_dim, v_dim, width, _ptr(mix), _ptr(norm_w), float(norm_eps), _ptr(cs_table),
+            int(rot), int(style), _ptr(v_first), 0 if v_first is None else v_first.stride(0), float(v_mix), _ptr(positions), _ptr(token_seq),
+            _ptr(block_table), block_table.shape[1], int(page_size), k_pages.shape[0], 1 if write_kv else 0, _ptr(q), _ptr(k_pages), _ptr(v_pages),
+            self._dt(proj), self._stream(proj)), "joint_qkv_store")
+        self.launches += 1
+        return q
+
+    def joint_plan(self, dtype, num_seqs, num_heads, kv_heads, width, v_dim, max_q_len, max_kv_len, page_size, keep_first=0):
+        """(kernel, num_splits, split_len) for attention over joint rows: a tensor-core kernel that sees one shared key head of
+        ``width`` values where one takes that width, else "joint", the general kernel."""
+        if dtype == torch.bfloat16 and (self.lib.ttie_attn_mma_supported(width)
+                                        or (width > 128 and self.lib.ttie_attn_tc_supported(width, page_size))):
+            return self.attention_plan(dtype, num_seqs, num_heads, 1, width, max_q_len, max_kv_len, page_size)
+        base = num_seqs * kv_heads * math.ceil(max_q_len * (num_heads // kv_heads) / self.lib.ttie_attn_joint_tile_rows(width, v_dim))
+        if base >= self.num_sms or max_kv_len <= 32:
+            return "joint", 1, 0
+        want = max(1, min(2 * self.num_sms // base, math.ceil(max_kv_len / 32)))
+        split_len = math.ceil(math.ceil(max_kv_len / want) / 32) * 32
+        n = math.ceil(max_kv_len / split_len)
+        return ("joint", n, split_len) if n > 1 else ("joint", 1, 0)
+
+    def paged_attention_joint(self, q, num_heads, kv_heads, width, v_dim, k_pages, v_pages, block_table, page_size, query_start_loc,
+                              seq_lens, num_seqs, max_q_len, max_kv_len, scale, window, out, chunk=0, keep_first=0, plan=None):
+        """Causal attention over joint rows: q [T, H * width] from ``joint_qkv_store``, pages [pages, 1, page, width]; head h's
+        output is its own kv head's value columns, out [T, H * v_dim]."""
+        T = q.shape[0]
+        if max_kv_len > block_table.shape[1] * page_size:
+            raise KernelError(f"paged_attention: a block table of {block_table.shape[1]} pages of {page_size} keys cannot cover {max_kv_len} keys")
+        kernel, num_splits, split_len = plan if plan is not None else self.joint_plan(
+            q.dtype, num_seqs, num_heads, kv_heads, width, v_dim, max_q_len, self.visible_keys(max_q_len, max_kv_len, window, chunk, keep_first),
+            page_size)
+        if kernel != "joint":
+            direct = kv_heads == 1 and v_dim == width
+            rows = out if direct else torch.empty((T, num_heads * width), dtype=q.dtype, device=q.device)
+            self.paged_attention(q, num_heads, 1, width, k_pages, v_pages, block_table, page_size, query_start_loc, seq_lens, num_seqs,
+                                 max_q_len, max_kv_len, scale, window, rows, plan=(kernel, num_splits, split_len), chunk=chunk, keep_first=keep_first)
+            if not direct:
+                self._check(self.lib.ttie_joint_values(_ptr(rows), _ptr(out), T, num_heads, kv_heads, v_dim, width, self._dt(q), self._stream(q)),
+                            "joint_values")
+                self.launches += 1
+            return
+        scratch = torch.empty((T * num_heads * num_splits * (v_dim + 2),), dtype=torch.float32, device=q.device) if num_splits > 1 else None
+        self._check(self.lib.ttie_paged_attention_joint(
+            _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1], page_size, _ptr(query_start_loc), _ptr(seq_lens),
+            _ptr(out), T, num_seqs, num_heads, kv_heads, width, v_dim, max_q_len, float(scale), int(window), int(chunk), int(keep_first),
+            num_splits, split_len, _ptr(scratch), self._dt(q), self._stream(q)), "paged_attention_joint")
         self.launches += 2 if num_splits > 1 else 1
 
     # ---- post-norm layers
@@ -973,16 +1089,20 @@ class CudaOps:
         return torch.bmm(x, w.transpose(1, 2))
 
     # ---- recurrent block
-    def causal_conv(self, xin, col0, width, taps, conv_w, conv_b, state, token_seq, query_start_loc, slot_ids, want_copy):
+    def causal_conv(self, xin, col0, width, taps, conv_w, conv_b, state, token_seq, query_start_loc, slot_ids, want_copy, first_row=1,
+                    act=None, want_f32=True):
         """Per-channel causal convolution over the step's tokens (``conv_w`` tap-major [taps, width]); inputs before the
-        step come from the state rows.
-        Returns (u float32 [T, width], u in the compute dtype or None)."""
+        step come from the state rows ``state`` [slots + 1, rows, width], whose rows from ``first_row`` on are the taps - 1 earlier
+        inputs, oldest first.  ``act`` "silu": applied to the sum.
+        Returns (u float32 [T, width] or None, u in the compute dtype or None)."""
         T = xin.shape[0]
-        u32 = torch.empty((T, width), dtype=torch.float32, device=xin.device)
+        u32 = torch.empty((T, width), dtype=torch.float32, device=xin.device) if want_f32 else None
         u_c = torch.empty((T, width), dtype=xin.dtype, device=xin.device) if want_copy else None
         self._check(self.lib.ttie_causal_conv(_ptr(xin), xin.stride(0), int(col0), T, width, taps, _ptr(conv_w), _ptr(conv_b),
-                                              self._dt(conv_w), _ptr(state), state.shape[0], _ptr(token_seq), _ptr(query_start_loc),
-                                              _ptr(slot_ids), _ptr(u32), _ptr(u_c), self._dt(xin), self._stream(xin)), "causal_conv")
+                                              self._dt(conv_w), _ptr(state), 0 if state is None else state.shape[0],
+                                              0 if state is None else state.stride(0), int(first_row) * width, {None: 0, "silu": 1}[act],
+                                              _ptr(token_seq), _ptr(query_start_loc), _ptr(slot_ids), _ptr(u32),
+                                              _ptr(u_c), self._dt(xin), self._stream(xin)), "causal_conv")
         self.launches += 1
         return u32, u_c
 
@@ -1007,10 +1127,52 @@ class CudaOps:
         self.launches += 4 if ws is not None else 1
         return out
 
+    # ---- selective scan
+    selective_warps = 12                    # warps per SM (4 schedulers) that a long prompt's scan is cut into parts for,
+    selective_max_parts = 16                # at most this many a request,
+    selective_part_tokens = 64              # of at least this many tokens
+
+    def selective_parts(self, num_tokens: int, num_seqs: int, channels: int, states: int) -> int:
+        """Into how many parts a request's tokens are walked: every part but the last is walked twice, which pays while the
+        channels alone give the SMs too few warps to hide a token's latency."""
+        longest = num_tokens - (num_seqs - 1)                          # the most tokens one request of the step can bring
+        pad = self.selective_state_pad(states)
+        lanes = pad // (4 if states <= 128 else 8 if states <= 256 else 16)
+        warps = num_seqs * -(-channels * lanes // 32)
+        return max(1, min(self.selective_max_parts, longest // self.selective_part_tokens, self.selective_warps * self.num_sms // warps))
+
+    @staticmethod
+    def selective_state_pad(states: int) -> int:
+        """States of a channel's row as the scan lays it out: a power-of-two number of slices of 4 (up to 128 states), 8 (up to
+        256) or 16."""
+        per_thread = 4 if states <= 128 else 8 if states <= 256 else 16
+        slices = 1
+        while slices * per_thread < states:
+            slices *= 2
+        return slices * per_thread
+
+    def selective_scan(self, u, dt, dt_bias, A, D, bc, col_b, col_c, z, state, xin, tail, taps, query_start_loc, slot_ids, num_seqs, states):
+        """The diagonal recurrence over the step's tokens from the state rows ``state`` [slots + 1, channels, padded states] (advanced
+        in place), with read-out, skip (``D``) and gate: returns (S C + D u) * silu(z) [T, channels] in the compute dtype.  ``u``,
+        ``z``: views [T, channels]; ``dt`` float32 [T, channels] before bias and softplus; ``A`` float32 [channels, padded states];
+        ``bc``: rows that hold B at column ``col_b`` and C at ``col_c``.  Also moves the last ``taps - 1`` rows of ``xin`` (the
+        convolution's inputs) into the state rows ``tail`` (None with one tap)."""
+        T, I = u.shape
+        out = torch.empty((T, I), dtype=u.dtype, device=u.device)
+        parts = self.selective_parts(T, int(num_seqs), I, int(states))
+        scratch = torch.empty(int(num_seqs) * parts * I * (A.shape[1] + 1), dtype=torch.float32, device=u.device) if parts > 1 else None
+        self._check(self.lib.ttie_selective_scan(
+            _ptr(u), u.stride(0), _ptr(dt), dt.stride(0), _ptr(dt_bias), _ptr(A), _ptr(D), _ptr(bc), bc.stride(0), int(col_b), int(col_c), _ptr(z),
+            z.stride(0), _ptr(state), state.shape[0], _ptr(xin), xin.stride(0), _ptr(tail), 0 if tail is None else tail.shape[0], int(taps),
+            _ptr(query_start_loc), _ptr(slot_ids), int(num_seqs), _ptr(out), I, int(states), parts, _ptr(scratch), self._dt(u), self._stream(u)),
+            "selective_scan")
+        self.launches += 2 if parts > 1 else 1
+        return out
+
     # ---- attention with a short convolution on its projections, partial rotation, another value size, gated heads
     def qkv_conv_rope_store(self, proj, num_heads, num_kv_heads, head_dim, v_dim, padded_dim, taps, conv_w, tail, positions, token_seq,
                             query_start_loc, slot_ids, cs_table, rot, style, k_pages, v_pages, block_table, page_size, write_kv,
-                            norm_w=None, norm_eps=0.0, v_from_k=False, q_temp=None, row_inv=None):
+                            norm_w=None, norm_eps=0.0, v_from_k=False, q_temp=None, row_inv=None, v_first=None, v_mix=0.0):
         """From a step's projected rows ``proj`` [T, >= Hq*D + Hkv*D + Hkv*Dv] (columns [q | k | v]): the short causal
         convolution over time (``conv_w`` float32 tap-major [taps, channels]; ``tail`` float32 state rows
         [slots + 1, taps - 1, channels] with each request's last projected rows; ``taps`` 1 and ``conv_w`` None: none), the
@@ -1022,6 +1184,7 @@ class CudaOps:
         ``q_temp`` (coef, every): q at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1).
         ``row_inv`` (float32 [T, 2] from ``proj_row_rms``): one norm over the whole q and one over the whole k projection
         instead of one per head; ``norm_w`` is then float32 [Hq*D + Hkv*D], a weight per channel.
+        ``v_first`` (a view [T, Hkv*Dv] with a row stride): values are stored as (1 - v_mix) * v + v_mix * v_first.
         Returns q [T, Hq * padded_dim].  The state rows are advanced by ``conv_tail_update``."""
         T = proj.shape[0]
         q = torch.empty((T, num_heads * padded_dim), dtype=proj.dtype, device=proj.device)
@@ -1030,6 +1193,7 @@ class CudaOps:
             0 if tail is None else tail.shape[0], _ptr(positions), _ptr(token_seq), _ptr(query_start_loc), _ptr(slot_ids),
             _ptr(cs_table), int(rot), int(style), _ptr(norm_w), float(norm_eps), _ptr(row_inv), 1 if v_from_k else 0,
             float(q_temp[0]) if q_temp else 0.0, int(q_temp[1]) if q_temp else 0,
+            _ptr(v_first), 0 if v_first is None else v_first.stride(0), float(v_mix),
             _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1],
             int(page_size), k_pages.shape[0], 1 if write_kv else 0, self._dt(proj), self._stream(proj)), "qkv_conv_rope_store")
         self.launches += 1
@@ -1198,14 +1362,24 @@ class CudaOps:
         return out
 
     # ---- elementwise functions between products
-    _ACTIVATIONS = {"relu2": 0, "tanh": 1, "softcap": 2}
+    _ACTIVATIONS = {"relu2": 0, "tanh": 1, "softcap": 2, "identity": 3, "silu": 4}
 
-    def activation(self, x, kind, out_dtype=None, c=0.0, inplace=False):
-        """f(x) elementwise in 32-bit: "relu2" (relu squared), "tanh", "softcap" (c * tanh(x / c)); x contiguous."""
+    def activation_rows(self, x, cols, kind, c=0.0, scale=1.0):
+        """f(x * scale) of the first ``cols`` columns of ``x`` (a view with a row stride) as contiguous float32 rows [T, cols]."""
+        T = x.shape[0]
+        out = torch.empty((T, cols), dtype=torch.float32, device=x.device)
+        self._check(self.lib.ttie_activation_rows(_ptr(x), x.stride(0), _ptr(out), T, int(cols), self._ACTIVATIONS[kind], float(c), float(scale),
+                                                  self._dt(x), self._stream(x)), "activation_rows")
+        self.launches += 1
+        return out
+
+    def activation(self, x, kind, out_dtype=None, c=0.0, inplace=False, scale=1.0):
+        """f(x * scale) elementwise in 32-bit: "relu2" (relu squared), "tanh", "softcap" (c * tanh(x / c)), "silu", "identity"; x
+        contiguous."""
         if not x.is_contiguous():
             raise KernelError("activation: the input must be contiguous")
         out = x if inplace else torch.empty(x.shape, dtype=out_dtype or x.dtype, device=x.device)
-        self._check(self.lib.ttie_activation(_ptr(x), _ptr(out), x.numel(), self._ACTIVATIONS[kind], float(c), self._dt(x),
+        self._check(self.lib.ttie_activation(_ptr(x), _ptr(out), x.numel(), self._ACTIVATIONS[kind], float(c), float(scale), self._dt(x),
                                              self._dt(out), self._stream(x)), "activation")
         self.launches += 1
         return out

@@ -31,10 +31,19 @@ only), ``qk_norm`` (its eps: every query and key head is divided by its root mea
 they are cut into heads, and a weight per channel, ``<q><norm_suffix>`` of ``heads * head_dim`` values and ``<k><norm_suffix>`` of
 ``kv_heads * head_dim``; the default ``"head"`` is the norm per head above), ``weights="sigmoid"`` (no softmax: a visible key
 weighs ``sigmoid(score + b_h)`` and the weights are not normalised over the keys; ``head_bias`` names the tensor of one ``b``
-per head, None: no bias).  The general step: one product
+per head, None: no bias), ``keep_first`` (with a window: a token also sees the sequence's first ``keep_first`` tokens, at their true
+positions), ``v_mix`` (``"first"``: this layer's values are kept for later layers of the step; ``"mix"``: the values become
+``(1 - l) v + l v_first`` with the number ``l`` of tensor ``v_mix_name`` and ``v_first`` the values of that first layer, and the mixed
+ones are cached), ``head_mix`` (the name of a matrix M [heads, heads]: head h's scores become ``sum_g M[h, g] score_g`` before the
+softmax; see below).  The general step: one product
 ``[W_q; W_k; W_v; W_g] x``; one kernel convolves, normalises, rotates, writes q and stores k and v - rows padded with zeros to
 ``padded_dim``, a multiple of 16 that holds both sizes, so every attention kernel of the package applies; a second moves the
 convolution's inputs into the state row; attention; the gate kernel drops the padding; ``W_o``.
+
+With ``head_mix`` the mixing goes into the queries: it is linear, so head h's mixed score is the product of ONE query row per head,
+``[sum of M[h, g] q_g over the heads g of kv head c]`` for every kv head c, with the keys of all kv heads side by side.  One kernel
+norms, rotates, mixes (32-bit) and stores; keys and values are cached as joint rows of all kv heads (one cache head); the
+attention kernels then see plain attention on one shared key head, and head h takes its own kv head's value columns.
 """
 from __future__ import annotations
 
@@ -57,7 +66,8 @@ class PagedAttention(Mixer):
                  gated=False, qkv_bias: bool = False, weight_suffix: str = ".weight", bias_suffix: str = ".bias",
                  conv_suffix: str = ".conv", chunk: Optional[int] = None, qk_norm: Optional[float] = None,
                  norm_suffix: str = ".norm", v_from_k: bool = False, q_temp: Optional[Dict[str, float]] = None,
-                 qk_norm_over: str = "head", weights: str = "softmax", head_bias: Optional[str] = None):
+                 qk_norm_over: str = "head", weights: str = "softmax", head_bias: Optional[str] = None, keep_first: int = 0,
+                 v_mix: Optional[str] = None, v_mix_name: str = "vmix", head_mix: Optional[str] = None):
         super().__init__(prefix)
         if num_heads % num_kv_heads:
             raise ValueError(f"num_heads={num_heads} is not a multiple of num_kv_heads={num_kv_heads}")
@@ -110,7 +120,20 @@ class PagedAttention(Mixer):
         self.rot_dim = int(getattr(self.position, "dim", 0) or 0)      # rotated values per head (0: none)
         if self.rot_dim > head_dim:
             raise ValueError(f"the position encoding rotates {self.rot_dim} values of a head of {head_dim}")
-        self.general = (self.v_head_dim != head_dim or self.has_conv or self.gated or self.qkv_bias
+        self.keep_first = int(keep_first or 0)
+        if self.keep_first < 0 or (self.keep_first and window is None):
+            raise ValueError(f"keep_first={keep_first} must not be negative and belongs to a window")
+        if v_mix not in (None, "first", "mix"):
+            raise ValueError(f"v_mix must be None, 'first' or 'mix', got {v_mix!r}")
+        if v_mix is not None and (self.v_from_k or conv_taps is not None):
+            raise ValueError("mixed values need a value projection without a convolution")
+        self.v_mix, self.v_mix_name, self.v_mix_weight = v_mix, v_mix_name, 0.0
+        self.head_mix, self.mix_t = head_mix, None
+        if head_mix is not None and (self.has_conv or self.gated or self.qkv_bias or self.v_from_k or self.q_temp is not None
+                                     or self.softcap is not None or self.weights != "softmax" or (self.qk_norm is not None and not self.norm_whole)):
+            raise ValueError("scores mixed over the heads exclude a convolution, gates, biases, keys as values, a query temperature, a "
+                             "score softcap, other weights than a softmax and a norm per head")
+        self.general = (self.v_head_dim != head_dim or self.v_mix is not None or self.head_mix is not None or self.has_conv or self.gated or self.qkv_bias
                         or self.rot_dim not in (0, head_dim) or self.qk_norm is not None or self.v_from_k
                         or self.q_temp is not None or self.weights != "softmax")
         if self.general and (self.shares_kv or self.bias):
@@ -118,6 +141,7 @@ class PagedAttention(Mixer):
         self.padded_dim = -(-max(head_dim, self.v_head_dim) // 16) * 16 if self.general else head_dim
         self.channels = (num_heads + num_kv_heads) * head_dim + (0 if self.v_from_k else num_kv_heads * self.v_head_dim)   # of [q | k | v]
         self.conv_w = self.norm_w = None
+        self.joint_dim = None                                           # values of a joint cache row (head_mix), set by validate
 
     def children(self):
         return [self.position]
@@ -153,6 +177,10 @@ class PagedAttention(Mixer):
         if self.qk_norm is not None:
             for key in ("q", "k"):
                 specs[f"{n[key]}{self.norm_suffix}"] = ParamSpec((rows[key] if self.norm_whole else D,), storage="vector", init="ones")
+        if self.v_mix is not None:                                     # (the first such layer's number is not used)
+            specs[self.v_mix_name] = ParamSpec((), storage="vector", init="normal", std=0.5)
+        if self.head_mix is not None:
+            specs[self.head_mix] = ParamSpec((self.num_heads, self.num_heads), storage="vector", init="normal", std=0.3)
         if self.head_bias_name is not None:
             specs[self.head_bias_name] = ParamSpec((self.num_heads,), storage="vector", init="normal", std=0.5)
         if self.gated:
@@ -176,6 +204,10 @@ class PagedAttention(Mixer):
         if self.qk_norm is not None:                                    # 32-bit, the query heads' weights then the key heads'
             ws_ = [params[f"{n[k]}{self.norm_suffix}"].float() for k in ("q", "k")]
             self.norm_w = (torch.cat(ws_) if self.norm_whole else torch.stack(ws_)).contiguous()
+        if self.v_mix == "mix":
+            self.v_mix_weight = float(params[self.v_mix_name].float().item())
+        if self.head_mix is not None:                                   # transposed, 32-bit: the weights of one source head lie side by side
+            self.mix_t = params[self.head_mix].float().t().contiguous()
         if self.head_bias_name is not None:
             self.head_bias = params[self.head_bias_name].float().contiguous()
 
@@ -194,18 +226,65 @@ class PagedAttention(Mixer):
         return [self.w_in, self.w_out]
 
     def validate(self, ops, dtype, page_size):
+        if self.head_mix is not None:
+            ops.check_joint_attention(dtype, self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim, self.page_size or page_size)
+            self.joint_dim = ops.joint_width(dtype, self.num_kv_heads, self.head_dim, self.v_head_dim)
+            return
         check = getattr(ops, "check_attention", None)
         if check is not None:
             check(dtype, self.num_heads, self.num_kv_heads, self.padded_dim, self.page_size or page_size)
 
     # ---------------------------------------------------------------- cache
     def cache_needs(self):
-        needs = [PagedKVNeed(self.num_kv_heads, self.padded_dim, self.window, self.page_size, chunk=self.chunk)]
+        if self.head_mix is not None:                                   # joint rows: one cache head (its width: validate, or unpadded)
+            width = self.joint_dim or self.num_kv_heads * max(self.head_dim, self.v_head_dim)
+            return [PagedKVNeed(1, width, self.window, self.page_size, chunk=self.chunk, keep_first=self.keep_first)]
+        needs = [PagedKVNeed(self.num_kv_heads, self.padded_dim, self.window, self.page_size, chunk=self.chunk, keep_first=self.keep_first)]
         if self.conv_taps > 1:
             needs.append(FixedStateNeed((self.conv_taps - 1, self.channels), "float32"))
         return needs
 
     # ---------------------------------------------------------------- step
+    def _first_values(self, v, ctx):
+        """The values that this layer's are mixed with (None: not mixed); the first such layer of a step leaves its own."""
+        if self.v_mix is None:
+            return None
+        key = ("first values", self.v_mix_name)
+        if self.v_mix == "first":
+            ctx.step_cache[key] = v
+            return None
+        return ctx.step_cache[key]
+
+    def _joint_forward(self, x, ctx, cache):
+        ops = self.ops
+        H, G, D, Dv, W = self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim, self.joint_dim
+        proj = ops.linear(x, self.w_in, None)                        # [T, q | k | v]
+        table = self.position.rotary_table()
+        inv_freq, style = table if table is not None else (None, 0)
+        rot = self.rot_dim if inv_freq is not None else 0
+        cs = self.position.step_table(ctx) if rot else None
+        v_first = self._first_values(proj[:, (H + G) * D:], ctx)
+        q = ops.joint_qkv_store(proj, H, G, D, Dv, W, self.mix_t, ctx.positions, ctx.token_seq, cs, rot, style, cache.k_pages, cache.v_pages,
+                                cache.block_table, cache.page_size, cache.writable, norm_w=self.norm_w, norm_eps=self.qk_norm or 0.0,
+                                v_first=v_first, v_mix=self.v_mix_weight)
+        out = torch.empty((proj.shape[0], H * Dv), dtype=x.dtype, device=x.device)
+        classes = ctx.classes()
+        for ci, c in enumerate(classes):
+            views = (cache.block_table, ctx.seq_lens) if len(classes) == 1 else self._class_views(ctx, cache, ci, c)
+            ops.paged_attention_joint(q[c.tok_lo:c.tok_hi], H, G, W, Dv, cache.k_pages, cache.v_pages, views[0], cache.page_size,
+                                      c.query_start_loc, views[1], c.seq_hi - c.seq_lo, c.max_q_len, c.max_kv_len, self.scale, self.window or 0,
+                                      out[c.tok_lo:c.tok_hi], chunk=self.chunk or 0, keep_first=self.keep_first)
+        return ops.linear(out, self.w_out, None, partial_ok=True)
+
+    @staticmethod
+    def _class_views(ctx, cache, ci, c):
+        """The block table and lengths of one class of the step's requests: the same for every layer of a cache group."""
+        key = ("attention class views", id(cache.block_table), ci)
+        views = ctx.step_cache.get(key)
+        if views is None:
+            views = ctx.step_cache[key] = (cache.block_table[c.seq_lo:c.seq_hi], ctx.seq_lens[c.seq_lo:c.seq_hi])
+        return views
+
     def _general_forward(self, x, ctx, cache, tail):
         ops = self.ops
         Hq, Hkv, D, Dv, Dp, C = self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim, self.padded_dim, self.channels
@@ -216,11 +295,13 @@ class PagedAttention(Mixer):
         rot = self.rot_dim if inv_freq is not None else 0
         cs = self.position.step_table(ctx) if rot else None
         state = tail.state if tail is not None else None
+        v_first = self._first_values(proj[:, (Hq + Hkv) * D:C], ctx)
+        mixed = {} if v_first is None else {"v_first": v_first, "v_mix": self.v_mix_weight}
         row_inv = ops.proj_row_rms(proj, Hq * D, Hkv * D, self.qk_norm) if self.norm_whole else None
         q = ops.qkv_conv_rope_store(proj, Hq, Hkv, D, Dv, Dp, self.conv_taps, self.conv_w, state, ctx.positions, ctx.token_seq,
                                     ctx.query_start_loc, ctx.slot_ids, cs, rot, style, cache.k_pages, cache.v_pages,
                                     cache.block_table, cache.page_size, cache.writable, norm_w=self.norm_w,
-                                    norm_eps=self.qk_norm or 0.0, v_from_k=self.v_from_k, q_temp=self.q_temp, row_inv=row_inv)
+                                    norm_eps=self.qk_norm or 0.0, v_from_k=self.v_from_k, q_temp=self.q_temp, row_inv=row_inv, **mixed)
         if self.conv_taps > 1 and tail.writable:
             ops.conv_tail_update(proj, C, self.conv_taps, state, ctx.query_start_loc, ctx.slot_ids, ctx.num_seqs)
         out = torch.empty((T, Hq * Dp), dtype=x.dtype, device=x.device)
@@ -233,6 +314,8 @@ class PagedAttention(Mixer):
         """One attention launch per class of requests (decoded tokens; prompt portions), each planned as if it were alone."""
         ops, Hq, Hkv = self.ops, self.num_heads, self.num_kv_heads
         extra = {} if self.weights == "softmax" else {"weights": self.weights, "head_bias": self.head_bias}
+        if self.keep_first:
+            extra["keep_first"] = self.keep_first
         classes = ctx.classes()
         if len(classes) == 1:
             c = classes[0]
@@ -241,10 +324,7 @@ class PagedAttention(Mixer):
                                 self.scale, self.window or 0, out, softcap=self.softcap or 0.0, chunk=self.chunk or 0, **extra)
             return
         for ci, c in enumerate(classes):
-            key = ("attention class views", id(cache.block_table), ci)    # the same for every layer of a cache group
-            views = ctx.step_cache.get(key)
-            if views is None:
-                views = ctx.step_cache[key] = (cache.block_table[c.seq_lo:c.seq_hi], ctx.seq_lens[c.seq_lo:c.seq_hi])
+            views = self._class_views(ctx, cache, ci, c)
             ops.paged_attention(q[c.tok_lo:c.tok_hi], Hq, Hkv, D, cache.k_pages, cache.v_pages, views[0],
                                 cache.page_size, c.query_start_loc, views[1], c.seq_hi - c.seq_lo, c.max_q_len,
                                 c.max_kv_len, self.scale, self.window or 0, out[c.tok_lo:c.tok_hi], softcap=self.softcap or 0.0,
@@ -255,6 +335,8 @@ class PagedAttention(Mixer):
         if isinstance(cache, (list, tuple)):                         # the views in the order of cache_needs()
             tail = cache[1] if len(cache) > 1 else None
             cache = cache[0]
+        if self.head_mix is not None:
+            return self._joint_forward(x, ctx, cache)
         if self.general:
             return self._general_forward(x, ctx, cache, tail)
         ops = self.ops

@@ -9,7 +9,8 @@ view the cache manager made for it.
 
 Categories and the methods each must have:
 
-``norm``      ``add_norm(resid, delta) -> x``; ``norm_rows(resid, delta, rows) -> x`` (post-norm blocks: ``scale_add_norm``)
+``norm``      ``add_norm(resid, delta) -> x``; ``norm_rows(resid, delta, rows) -> x`` (post-norm blocks: ``scale_add_norm``;
+              both take ``delta_norm``, a norm the delta passes before it is added, where a block leaves one)
 ``position``  ``rotary_table() -> (inv_freq, style) | None``; ``apply(q, k, positions)``
 ``mixer``     ``cache_need()`` (or ``cache_needs()`` for several); ``forward(x, ctx, cache) -> y``
 ``ffn``       ``forward(x, ctx) -> y``
@@ -94,6 +95,7 @@ class PagedKVNeed:
     page_size: Optional[int] = None    # None: the engine's page size
     planes: int = 2                    # 2: keys and values; 1: one array that is both (latent attention), handed out as K and as V
     chunk: Optional[int] = None        # a token reads only keys of its own chunk (chunks counted from position 0); excludes window
+    keep_first: int = 0                # with a window: the sequence's first tokens that every later one still reads
 
 
 @dataclass(frozen=True)
@@ -177,14 +179,17 @@ class ResidualStream:
     """The residual sum in 32-bit plus the last sub-layer's output not yet added to it.
 
     Norm parts add ``delta`` into ``resid`` in the same kernel that normalises, so the
-    sum is formed and kept in 32-bit whatever the compute dtype is.  ``x`` (post-norm blocks): a copy of
-    ``resid`` in the compute dtype, if a norm kernel has written one (sub-layers there read the stream itself).
+    sum is formed and kept in 32-bit whatever the compute dtype is.  ``delta_norm``: a norm part that the
+    waiting output passes before it is added (blocks that norm a sub-layer's output as well as its input), or None.
+    ``x`` (post-norm blocks): a copy of ``resid`` in the compute dtype, if a norm kernel has written one (sub-layers
+    there read the stream itself).
     """
-    __slots__ = ("resid", "delta", "x")
+    __slots__ = ("resid", "delta", "delta_norm", "x")
 
     def __init__(self, resid: torch.Tensor, delta: Optional[torch.Tensor] = None):
         self.resid = resid
         self.delta = delta
+        self.delta_norm = None
         self.x = None
 
 
@@ -228,11 +233,11 @@ class Part:
 class Norm(Part):
     category = "norm"
 
-    def add_norm(self, resid: torch.Tensor, delta: Optional[torch.Tensor]) -> torch.Tensor:
+    def add_norm(self, resid: torch.Tensor, delta: Optional[torch.Tensor], delta_norm: Optional["Norm"] = None) -> torch.Tensor:
         raise NotImplementedError
 
     def norm_rows(self, resid: torch.Tensor, delta: Optional[torch.Tensor], rows: torch.Tensor,
-                  num_rows: int) -> torch.Tensor:
+                  num_rows: int, delta_norm: Optional["Norm"] = None) -> torch.Tensor:
         raise NotImplementedError
 
 

@@ -32,13 +32,47 @@ class PreNormBlock(Block):
         return self.mixer.cache_needs()                            # the feed-forward parts here keep nothing between steps
 
     def forward(self, stream: ResidualStream, ctx: StepContext, caches) -> None:
-        h = self.mixer_norm.add_norm(stream.resid, stream.delta)
+        pending = {} if stream.delta_norm is None else {"delta_norm": stream.delta_norm}
+        h = self.mixer_norm.add_norm(stream.resid, stream.delta, **pending)
+        stream.delta_norm = None
         a = self.mixer.forward(h, ctx, mixer_cache_argument(self.mixer, caches))
         if self.ffn is None:
             stream.delta = a
             return
         h = self.ffn_norm.add_norm(stream.resid, a)
         stream.delta = self.ffn.forward(h, ctx)
+
+
+@register_part("block", "sandwich_norm")
+class SandwichNormBlock(Block):
+    """A norm before and a norm after each sub-layer: ``x = x + norm_b(mixer(norm_a(x)))`` followed by
+    ``x = x + norm_d(ffn(norm_c(x)))``.  A sub-layer's output waits unnormed in ``stream.delta`` with its norm in
+    ``stream.delta_norm``; the next norm applies that one, adds, and normalises, in one kernel.  A layer without a feed-forward
+    (``ffn`` None) ends after the first sum."""
+
+    def __init__(self, prefix: str, mixer_norm: PartSpec, mixer: PartSpec, mixer_out_norm: PartSpec, ffn_norm: PartSpec = None,
+                 ffn: PartSpec = None, ffn_out_norm: PartSpec = None):
+        super().__init__(prefix)
+        self.mixer_norm = build_part("norm", mixer_norm)
+        self.mixer = build_part("mixer", mixer)
+        self.mixer_out_norm = build_part("norm", mixer_out_norm)
+        has = ffn is not None
+        self.ffn_norm = build_part("norm", ffn_norm) if has else None
+        self.ffn = build_part("ffn", ffn) if has else None
+        self.ffn_out_norm = build_part("norm", ffn_out_norm) if has else None
+
+    def children(self):
+        return [p for p in (self.mixer_norm, self.mixer, self.mixer_out_norm, self.ffn_norm, self.ffn, self.ffn_out_norm) if p is not None]
+
+    def cache_needs(self):
+        return self.mixer.cache_needs()
+
+    def forward(self, stream: ResidualStream, ctx: StepContext, caches) -> None:
+        h = self.mixer_norm.add_norm(stream.resid, stream.delta, stream.delta_norm)
+        stream.delta, stream.delta_norm = self.mixer.forward(h, ctx, mixer_cache_argument(self.mixer, caches)), self.mixer_out_norm
+        if self.ffn is not None:
+            h = self.ffn_norm.add_norm(stream.resid, stream.delta, stream.delta_norm)
+            stream.delta, stream.delta_norm = self.ffn.forward(h, ctx), self.ffn_out_norm
 
 
 @register_part("block", "post_norm")

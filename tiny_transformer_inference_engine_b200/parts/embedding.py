@@ -40,11 +40,11 @@ class TokenEmbedding(Embedding):
 
 @register_part("head", "linear")
 class LinearHead(Head):
-    """``logits = W x``; with ``softcap`` c the logits leave as ``c * tanh(logits / c)``.  ``name``: the matrix's relative name."""
+    """``logits = scale * W x``; with ``softcap`` c the logits leave as ``c * tanh(logits / c)``.  ``name``: the matrix's relative name."""
 
-    def __init__(self, prefix: str, dim: int, vocab_size: int, name: str = "weight", softcap=None):
+    def __init__(self, prefix: str, dim: int, vocab_size: int, name: str = "weight", softcap=None, scale: float = 1.0):
         super().__init__(prefix)
-        self.dim, self.vocab_size, self.name = int(dim), int(vocab_size), name
+        self.dim, self.vocab_size, self.name, self.scale = int(dim), int(vocab_size), name, float(scale)
         self.softcap = None if softcap is None else float(softcap)
         if self.softcap is not None and not self.softcap > 0:
             raise ValueError(f"softcap must be positive or None, got {softcap}")
@@ -62,7 +62,10 @@ class LinearHead(Head):
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         logits = self.ops.linear(x, self.weight, None, out_dtype=torch.float32)
         if self.softcap is not None:
-            self.ops.activation(logits, "softcap", c=self.softcap, inplace=True)
+            scale = {} if self.scale == 1.0 else {"scale": self.scale}
+            self.ops.activation(logits, "softcap", c=self.softcap, inplace=True, **scale)
+        elif self.scale != 1.0:
+            self.ops.activation(logits, "identity", inplace=True, scale=self.scale)
         return logits
 
 

@@ -5,6 +5,10 @@ Formula of the reference (models/rmsnorm.py:12-18): ``x32 = float(x)``,
 eps inside the square root, weight multiplied in 32-bit before the cast.  The
 reference fixes eps in code (models/rmsnorm.py:7) and never passes
 ``ModelConfig.rms_norm_eps``; here eps is this part's parameter.
+
+``scalar=True``: the weight is a single number for all coordinates (a tensor of shape []); it is spread over the width when it
+is loaded, so the kernels know one form.  ``delta_norm`` (another ``RMSNorm`` of the same width): the sub-layer's output passes
+that norm before it is added, in the same kernel: ``x += rms(delta) * w_d``, then ``rms(x) * w``.
 """
 from __future__ import annotations
 
@@ -18,32 +22,47 @@ from ..registry import register_part
 
 @register_part("norm", "rmsnorm")
 class RMSNorm(Norm):
-    def __init__(self, prefix: str, dim: int, eps: float, name: str = "weight"):
+    def __init__(self, prefix: str, dim: int, eps: float, name: str = "weight", scalar: bool = False):
         super().__init__(prefix)
         self.dim = int(dim)
         self.eps = float(eps)
         self.name = name                   # relative name of the weight tensor
+        self.scalar = bool(scalar)         # one number for all coordinates
         self.weight = None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
-        return {self.name: ParamSpec((self.dim,), storage="vector", init="ones")}
+        return {self.name: ParamSpec(() if self.scalar else (self.dim,), storage="vector", init="ones")}
 
     def load(self, params):
-        self.weight = params[self.name]
+        w = params[self.name]
+        self.weight = w.float().expand(self.dim).contiguous() if self.scalar else w
+        self._weight32 = None
+
+    @property
+    def weight32(self) -> torch.Tensor:
+        """The weight in 32-bit (what the two-norm kernel takes)."""
+        if self._weight32 is None:
+            self._weight32 = self.weight.float().contiguous()
+        return self._weight32
 
     def validate(self, ops, dtype, page_size):
         check = getattr(ops, "check_norm", None)
         if check is not None:
             check(dtype, self.dim)
 
-    def add_norm(self, resid: torch.Tensor, delta: Optional[torch.Tensor]) -> torch.Tensor:
+    def add_norm(self, resid: torch.Tensor, delta: Optional[torch.Tensor], delta_norm: Optional["RMSNorm"] = None) -> torch.Tensor:
         out = torch.empty(resid.shape, dtype=self.dtype, device=resid.device)
+        if delta_norm is not None and delta is not None:
+            self.ops.sandwich_norm(resid, delta, delta_norm.weight32, delta_norm.eps, self.weight32, self.eps, out)
+            return out
         self.ops.add_rmsnorm(resid, delta, self.weight, self.eps, out)
         return out
 
-    def norm_rows(self, resid, delta, rows, num_rows) -> torch.Tensor:
+    def norm_rows(self, resid, delta, rows, num_rows, delta_norm: Optional["RMSNorm"] = None) -> torch.Tensor:
         out = torch.empty((num_rows, self.dim), dtype=self.dtype, device=resid.device)
-        if num_rows:
+        if num_rows and delta_norm is not None and delta is not None:
+            self.ops.sandwich_norm(resid, delta, delta_norm.weight32, delta_norm.eps, self.weight32, self.eps, out, rows=rows, num_rows=num_rows)
+        elif num_rows:
             self.ops.rmsnorm_rows(resid, delta, rows, num_rows, self.weight, self.eps, out)
         return out
 

@@ -6,6 +6,11 @@ with the state S [dim x vdim] starting at zero,
 
     S_t = decay_h S_(t-1) + k_t v_t^T          o_t = S_t^T q_t
 
+Options, for relatives of it: ``qkv_act="silu"`` (q, k and v pass that activation behind their projections; no position encoding
+then), ``key_scale`` (what k is multiplied by; None: ``dim^(-1/2)``), ``norm_over="all"`` (one root mean square over the
+concatenated heads instead of one per head), ``norm_weight`` (the relative name of a weight per value behind the norm; None: no
+weight), ``gate_act`` (``"silu"`` or ``"sigmoid"``).
+
 Each head's ``o`` is divided by its root mean square (``x / sqrt(mean(x^2) + eps)``, no weight), the heads are concatenated,
 multiplied by ``silu(W_g h)`` and projected by ``W_o``.
 
@@ -28,7 +33,8 @@ from ..registry import register_part, build_part
 @register_part("mixer", "retention")
 class Retention(Mixer):
     def __init__(self, prefix: str, d_model: int, num_heads: int, dim: int, vdim: int, decay: Sequence[float], eps: float,
-                 position: Optional[PartSpec] = None, gate_act: str = "silu", names: Optional[Dict[str, str]] = None):
+                 position: Optional[PartSpec] = None, gate_act: str = "silu", names: Optional[Dict[str, str]] = None,
+                 qkv_act: Optional[str] = None, key_scale: Optional[float] = None, norm_over: str = "head", norm_weight: Optional[str] = None):
         super().__init__(prefix)
         self.d_model, self.num_heads, self.dim, self.vdim, self.eps = int(d_model), int(num_heads), int(dim), int(vdim), float(eps)
         self.decay = tuple(float(x) for x in decay)
@@ -43,24 +49,39 @@ class Retention(Mixer):
         self.rot_dim = int(getattr(self.position, "dim", 0) or 0)
         if self.rot_dim > self.dim:
             raise ValueError(f"retention: the position encoding rotates {self.rot_dim} values of a head of {self.dim}")
+        if qkv_act not in (None, "silu"):
+            raise ValueError(f"retention: unknown activation {qkv_act!r} on q, k and v")
+        if qkv_act is not None and self.rot_dim:
+            raise ValueError("retention: an activation on q, k and v and a position encoding exclude each other")
+        if norm_over not in ("head", "all"):
+            raise ValueError(f"retention: norm_over must be 'head' or 'all', got {norm_over!r}")
+        self.qkv_act, self.norm_over, self.norm_name = qkv_act, norm_over, norm_weight
+        self.key_scale = self.dim ** -0.5 if key_scale is None else float(key_scale)
+        if qkv_act is not None and self.key_scale != 1.0:
+            raise ValueError("retention: activated keys enter unscaled")
         self.names = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o"}
         if names:
             self.names.update(names)
-        self.w_in = self.w_out = self.decay_t = None
+        self.w_in = self.w_out = self.decay_t = self.norm_w = None
 
     def children(self):
         return [self.position]
 
     def param_specs(self):
         n, d, H, D, Dv = self.names, self.d_model, self.num_heads, self.dim, self.vdim
-        return {n["q"]: ParamSpec((H * D, d)), n["k"]: ParamSpec((H * D, d)), n["v"]: ParamSpec((H * Dv, d)),
-                n["g"]: ParamSpec((H * Dv, d)), n["o"]: ParamSpec((d, H * Dv))}
+        specs = {n["q"]: ParamSpec((H * D, d)), n["k"]: ParamSpec((H * D, d)), n["v"]: ParamSpec((H * Dv, d)),
+                 n["g"]: ParamSpec((H * Dv, d)), n["o"]: ParamSpec((d, H * Dv))}
+        if self.norm_name is not None:
+            specs[self.norm_name] = ParamSpec((H * Dv,), storage="vector", init="ones")
+        return specs
 
     def load(self, params):
         n = self.names
         self.w_in = torch.cat([params[n[s]] for s in ("q", "k", "v", "g")], dim=0).contiguous()       # [2*H*dim + 2*H*vdim, d]
         self.w_out = params[n["o"]].contiguous()
         self.decay_t = torch.tensor(self.decay, dtype=torch.float32, device=self.w_in.device)
+        if self.norm_name is not None:
+            self.norm_w = params[self.norm_name].float().contiguous()
 
     def product_weights(self):
         return [self.w_in, self.w_out]
@@ -72,13 +93,18 @@ class Retention(Mixer):
         ops, H, D, Dv = self.ops, self.num_heads, self.dim, self.vdim
         S = cache[0]
         proj = ops.linear(x, self.w_in, None)                                                  # [T, q | k | v | g]
-        table = self.position.rotary_table()
-        inv_freq, style = table if table is not None else (None, 0)
-        rot = self.rot_dim if inv_freq is not None else 0
-        cs = self.position.step_table(ctx) if rot else None
-        qk = ops.rotate_heads(proj, 2 * H, D, cs, rot, style, scale_from=H, scale=D ** -0.5)   # float32 [T, q | k]
         v, g = proj[:, 2 * H * D:2 * H * D + H * Dv], proj[:, 2 * H * D + H * Dv:]
-        o = ops.retention_scan(qk[:, :H * D], qk[:, H * D:], v, self.decay_t, S.state, ctx.query_start_loc, ctx.slot_ids,
+        if self.qkv_act is not None:                                                           # float32 [T, q | k | v]
+            qk = ops.activation_rows(proj, 2 * H * D + H * Dv, self.qkv_act)
+            v = qk[:, 2 * H * D:]
+        else:
+            table = self.position.rotary_table()
+            inv_freq, style = table if table is not None else (None, 0)
+            rot = self.rot_dim if inv_freq is not None else 0
+            cs = self.position.step_table(ctx) if rot else None
+            qk = ops.rotate_heads(proj, 2 * H, D, cs, rot, style, scale_from=H, scale=self.key_scale)   # float32 [T, q | k]
+        o = ops.retention_scan(qk[:, :H * D], qk[:, H * D:2 * H * D], v, self.decay_t, S.state, ctx.query_start_loc, ctx.slot_ids,
                                ctx.num_seqs, H, D, Dv)
-        y = ops.head_norm_gate(o, g, None, H, Dv, self.eps, self.gate_act)
+        heads, width = (1, H * Dv) if self.norm_over == "all" else (H, Dv)
+        y = ops.head_norm_gate(o, g, self.norm_w, heads, width, self.eps, self.gate_act)
         return ops.linear(y, self.w_out, None, partial_ok=True)
