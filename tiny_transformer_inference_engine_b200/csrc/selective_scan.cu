@@ -30,18 +30,20 @@ __device__ __forceinline__ int slot_row_(int slot, int num_rows) { return slot <
 __device__ __forceinline__ float softplusf_(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float siluf_(float x) { return x / (1.0f + expf(-x)); }
 
-// exp(dt * A).  A 32-bit run uses the library's function on A itself; a bfloat16 run the hardware's 2^x on A * log2(e), which
-// the thread holds instead (relative error about 1e-6, far below the rounding of the bfloat16 operands around it).
+// One step S <- exp(dt * A) S + x.  A slow state (dt * A near 0) lives for thousands of tokens, and the rounding of a factor just
+// below 1 repeats itself with every token: a 32-bit run adds expm1(dt * A) S + x to S instead, which leaves only the sum's own
+// rounding.  A bfloat16 run uses the hardware's 2^x on A * log2(e), which the thread then holds for A (relative error about
+// 2^-22, far below the rounding of the bfloat16 operands around it).
 template <typename T> struct Decay {
     static __device__ __forceinline__ float hold(float a) { return a; }
-    static __device__ __forceinline__ float of(float dt, float a) { return expf(dt * a); }
+    static __device__ __forceinline__ float step(float dt, float a, float S, float x) { return S + fmaf(expm1f(dt * a), S, x); }
 };
 template <> struct Decay<__nv_bfloat16> {
     static __device__ __forceinline__ float hold(float a) { return a * 1.4426950408889634f; }
-    static __device__ __forceinline__ float of(float dt, float a) {
+    static __device__ __forceinline__ float step(float dt, float a, float S, float x) {
         float y;
         asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(dt * a));
-        return y;
+        return fmaf(y, S, x);
     }
 };
 
@@ -117,8 +119,8 @@ __global__ void __launch_bounds__(NT) selective_scan_kernel(const SelArgs a) {
 #pragma unroll
             for (int i = 0; i < KPT; i += 4) {
                 const float4 x = *reinterpret_cast<const float4*>(add + i);
-                S[i] = fmaf(Decay<T>::of(sdt, Ah[i]), S[i], x.x); S[i + 1] = fmaf(Decay<T>::of(sdt, Ah[i + 1]), S[i + 1], x.y);
-                S[i + 2] = fmaf(Decay<T>::of(sdt, Ah[i + 2]), S[i + 2], x.z); S[i + 3] = fmaf(Decay<T>::of(sdt, Ah[i + 3]), S[i + 3], x.w);
+                S[i] = Decay<T>::step(sdt, Ah[i], S[i], x.x); S[i + 1] = Decay<T>::step(sdt, Ah[i + 1], S[i + 1], x.y);
+                S[i + 2] = Decay<T>::step(sdt, Ah[i + 2], S[i + 2], x.z); S[i + 3] = Decay<T>::step(sdt, Ah[i + 3], S[i + 3], x.w);
             }
         }
     }
@@ -139,7 +141,7 @@ __global__ void __launch_bounds__(NT) selective_scan_kernel(const SelArgs a) {
 #pragma unroll
             for (int i = 0; i < KPT; ++i) {
                 const bool in = n0 + i < a.N;
-                S[i] = fmaf(Decay<T>::of(dt, Ah[i]), S[i], du * (in ? to_f32(bp[(size_t)tt * a.ld_bc + n0 + i]) : 0.f));
+                S[i] = Decay<T>::step(dt, Ah[i], S[i], du * (in ? to_f32(bp[(size_t)tt * a.ld_bc + n0 + i]) : 0.f));
                 acc = fmaf(S[i], (in && !local) ? to_f32(cp[(size_t)tt * a.ld_bc + n0 + i]) : 0.f, acc);
             }
             sum_dt += dt;
@@ -199,8 +201,8 @@ __global__ void __launch_bounds__(NT) selective_scan_kernel(const SelArgs a) {
 #pragma unroll
                     for (int i = 0; i < KPT; i += 4) {
                         const float4 b = *reinterpret_cast<const float4*>(&b_s[tt][n0 + i]);
-                        S[i] = fmaf(Decay<T>::of(dt, Ah[i]), S[i], du * b.x); S[i + 1] = fmaf(Decay<T>::of(dt, Ah[i + 1]), S[i + 1], du * b.y);
-                        S[i + 2] = fmaf(Decay<T>::of(dt, Ah[i + 2]), S[i + 2], du * b.z); S[i + 3] = fmaf(Decay<T>::of(dt, Ah[i + 3]), S[i + 3], du * b.w);
+                        S[i] = Decay<T>::step(dt, Ah[i], S[i], du * b.x); S[i + 1] = Decay<T>::step(dt, Ah[i + 1], S[i + 1], du * b.y);
+                        S[i + 2] = Decay<T>::step(dt, Ah[i + 2], S[i + 2], du * b.z); S[i + 3] = Decay<T>::step(dt, Ah[i + 3], S[i + 3], du * b.w);
                         if (!local) {                                // (the same for every thread of the grid)
                             const float4 q = *reinterpret_cast<const float4*>(&c_s[tt][n0 + i]);
                             acc = fmaf(S[i], q.x, acc); acc = fmaf(S[i + 1], q.y, acc); acc = fmaf(S[i + 2], q.z, acc); acc = fmaf(S[i + 3], q.w, acc);
