@@ -349,8 +349,27 @@ def dabilorn_config(width, heads, layers=4):
             "max_seq_len": 4096}
 
 
+def renanex_config(width, heads, layers=4):
+    """A Renanex model at layer sizes that resemble a real model's: selective scan with twice the width as channels, 16 states, a
+    step-size rank of width / 16 and four convolution taps; linear attention with width / 128 heads of 128 key and 128 value
+    channels; attention with scores mixed over the heads, heads of 128 on one kv head (two from 16 heads on), YaRN-rescaled
+    rotation, a window of 1,024 keys that keeps the first four, and blended values; feed-forwards of 4 x width.  Layer order:
+    selective scan, linear attention, attention, attention, repeated."""
+    ssm = {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}
+    lin = {"heads": heads, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5 - 3 * i / max(1, heads - 1)) for i in range(heads)]}
+    att = {"heads": heads, "kv_heads": 2 if heads >= 16 else 1, "dim": 128, "vdim": 128, "mask": {"size": 1024, "keep_first": 4},
+           "rot": {"base": 10000.0, "dims": 128, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}},
+           "scale": 128 ** -0.5, "v_mix": True}
+    ff = {"kind": "dense", "ff": 4 * width}
+    kinds = (("mamba1", ssm), ("lightning", lin), ("attention", att), ("attention", att))
+    out = [{"type": kinds[i % 4][0], "mixer": dict(kinds[i % 4][1]), "mlp": ff} for i in range(layers)]
+    return {"architecture": "Renanex", "vocab": 32000, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 1.0, "logit_softcap": 30.0,
+            "layers": out, "max_seq_len": 4096}
+
+
 DESIGNS = {"munevik": ("Munevik", munevik_config, 1024), "mizupel": ("Mizupel", mizupel_config, 1024),
-           "mokalorn": ("Mokalorn", mokalorn_config, 0), "dabilorn": ("Dabilorn", dabilorn_config, 0)}     # name, configuration, window
+           "mokalorn": ("Mokalorn", mokalorn_config, 0), "dabilorn": ("Dabilorn", dabilorn_config, 0),
+           "renanex": ("Renanex", renanex_config, 1024)}     # name, configuration, window
 
 
 def like_config(width, heads, layers=4):
@@ -367,7 +386,7 @@ class OpRecorder:
              "rglru_scan", "glu", "linear_glu", "grouped_glu", "moe_route", "moe_plan", "grouped_linear", "moe_combine",
              "qkv_conv_rope_store", "conv_tail_update", "gate_head_rows", "token_shift_mix", "wkv_scan", "mlstm_scan", "head_norm_gate",
              "activation", "linear_act", "wkv_decay", "mlstm_gates", "rotate_heads", "retention_scan", "stream_conv", "proj_row_rms",
-             "rmsnorm_cols", "grouped_act")
+             "rmsnorm_cols", "grouped_act", "sandwich_norm", "joint_qkv_store", "paged_attention_joint", "selective_scan", "activation_rows", "linear_narrow")
 
     def __init__(self, ops):
         self.ops, self.calls, self.orig, self.depth = ops, [], {}, 0
@@ -426,6 +445,27 @@ def op_cost(name, args, kw, out, kv_lens, window):
         q, v, state, n, H, D, Dv = args[0], args[2], args[4], args[7], args[8], args[9], args[10]
         T = q.shape[0]
         return T * (2 * H * D * 4 + H * Dv * v.element_size() + 4 * H * Dv) + 2 * n * state[0].numel() * 4, ("fp32", 2 * T * 2 * H * D * Dv)
+    if name == "selective_scan":                                   # (u, dt, ..., A, D, bc, ..., z, state, ..., requests, states): an exponential and three multiply-adds per state and token
+        u, bc, z, S, n, N = args[0], args[5], args[8], args[9], args[15], args[16]
+        T, I = u.shape
+        return T * (3 * I * u.element_size() + 4 * I + bc.shape[1] * bc.element_size()) + 2 * n * I * N * 4, ("fp32", 2 * T * 3 * I * N)
+    if name == "sandwich_norm":                                    # (resid, delta, ...): the stream read and written (gathered rows: read), the delta read, one row out
+        rows = kw.get("num_rows") or args[0].shape[0]
+        per = args[0].shape[1] * ((4 if kw.get("rows") is not None else 8) + args[6].element_size())
+        return rows * per + _tensor_bytes(args[1]) * rows // args[0].shape[0], 0
+    if name == "activation_rows":                                  # (x, cols, ...)
+        return args[0].shape[0] * args[1] * args[0].element_size() + _tensor_bytes(out), 0
+    if name == "joint_qkv_store":                                  # the projected row read, joint query rows written, joint key and value rows stored
+        T, H, W = args[0].shape[0], args[1], args[5]
+        used = H * args[3] + args[2] * (args[3] + args[4])
+        es = args[0].element_size()
+        return T * es * (used + 2 * W) + _tensor_bytes(out), ("fp32", 2 * T * H * H * args[3])
+    if name == "paged_attention_joint":                            # plain grouped attention's bytes and products, and the mixing of the scores (H x H per key)
+        q, H, G, W, Dv, kp = args[0], args[1], args[2], args[3], args[4], args[5]
+        D, keep = W // G, kw.get("keep_first") or 0
+        seen = sum(sum(min(p + 1, (window or p + 1) + keep) for p in range(L - n, L)) for L, n in kv_lens)
+        vis = sum(min(L, (window + n + keep) if window else L) for L, n in kv_lens)
+        return (q.shape[0] * H * (D + Dv) + vis * G * (D + Dv)) * q.element_size(), seen * H * (2 * D + 2 * Dv + 2 * H)
     if name == "rotate_heads":                                     # (src, heads, dim, ...): the rotated columns read, 32-bit rows written
         return args[0].shape[0] * args[1] * args[2] * args[0].element_size() + _tensor_bytes(out), 0
     if name == "qkv_conv_rope_store":                              # pages and state rows are pools: count the rows read and written
@@ -438,7 +478,7 @@ def op_cost(name, args, kw, out, kv_lens, window):
         return _tensor_bytes([args[0], out]), 0
     if name in ("head_norm_gate", "gate_head_rows"):
         return _tensor_bytes([args[0], args[1], out]), 0
-    if name in ("linear", "linear_swiglu", "linear_glu", "linear_act"):
+    if name in ("linear", "linear_swiglu", "linear_glu", "linear_act", "linear_narrow"):
         x, w = args[0], args[1]
         flops = 2 * x.shape[0] * w.shape[0] * w.shape[1]
         return _tensor_bytes([x, w, out]), flops
@@ -503,7 +543,7 @@ def time_ops(eng, entries_fn, pk, kv_lens, window, iters=8):
         else:
             ideal = max(b / (pk["hbm_gbs"] * 1e9), f / (pk["bf16_tflops"] * 1e12)) * 1e6
         key = name
-        if name in ("linear", "batched_linear", "grouped_linear", "linear_swiglu", "linear_glu", "grouped_glu", "linear_act", "grouped_act"):
+        if name in ("linear", "batched_linear", "grouped_linear", "linear_swiglu", "linear_glu", "grouped_glu", "linear_act", "grouped_act", "linear_narrow"):
             w = args[1]
             key = f"{name} {list(w.shape)}"
         r = rows.setdefault(key, {"calls": 0, "us": 0.0, "ideal_us": 0.0})
@@ -587,8 +627,8 @@ def run_design(args, pk):
 
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default=None, choices=("munevik", "mizupel", "mokalorn", "dabilorn"), help="prefill and decode of this design at a few sizes beside the closest existing model, with per-operation times")
-    ap.add_argument("--beside", default=None, choices=("mqa_gpt", "munevik", "mizupel", "mokalorn", "dabilorn"), help="with --design: the model it is timed beside (default: the multi-query GPT)")
+    ap.add_argument("--design", default=None, choices=("munevik", "mizupel", "mokalorn", "dabilorn", "renanex"), help="prefill and decode of this design at a few sizes beside the closest existing model, with per-operation times")
+    ap.add_argument("--beside", default=None, choices=("mqa_gpt", "munevik", "mizupel", "mokalorn", "dabilorn", "renanex"), help="with --design: the model it is timed beside (default: the multi-query GPT)")
     ap.add_argument("--sizes", default=None, help="with --design: comma-separated model widths (multiples of 128)")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=64)

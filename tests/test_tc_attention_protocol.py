@@ -36,7 +36,7 @@ class Deadlock(Exception):
     pass
 
 
-def simulate(nsteps, ntq, seed, product_barriers_per_tile=2, softmax_threads=2, correction_threads=2):
+def simulate(nsteps, ntq, seed, product_barriers_per_tile=2, softmax_threads=2, correction_threads=2, NS=NS, KE=1):
     """One CTA walking `nsteps` key steps with `ntq` query tiles.  Raises AssertionError when a role touches data of
     the wrong step and Deadlock when nothing can move."""
     rnd = random.Random(seed)
@@ -66,17 +66,17 @@ def simulate(nsteps, ntq, seed, product_barriers_per_tile=2, softmax_threads=2, 
         return (("OF", t, j % PB), ((j // PB) & 1))
 
     def k_index(j):
-        return j if j < 2 else 2 * j - 1
+        return KE * j if j < 2 else 2 * KE + (KE + 1) * (j - 2) + 1
 
     def v_index(j):
-        return 2 * nsteps - 1 if j == nsteps - 1 else 2 * j + 2
+        return (KE + 1) * nsteps - 1 if j == nsteps - 1 else 2 * KE + (KE + 1) * j
 
     def producer():
-        order = [("K", 0)] + ([("K", 1)] if nsteps > 1 else [])
+        order = [("K", 0)] * KE + ([("K", 1)] * KE if nsteps > 1 else [])
         for j in range(nsteps):
             order.append(("V", j))
             if j + 2 < nsteps:
-                order.append(("K", j + 2))
+                order += [("K", j + 2)] * KE
         for it, tile in enumerate(order):
             st = it % NS
             yield from wait(("EMPTY", st), ((it // NS) & 1) ^ 1)
@@ -84,16 +84,18 @@ def simulate(nsteps, ntq, seed, product_barriers_per_tile=2, softmax_threads=2, 
 
     def score_issuer():
         for j in range(nsteps):
-            b, idx = j & 1, k_index(j)
-            st = idx % NS
-            yield from wait(("FULL", st), (idx // NS) & 1)
-            assert ring[st] == ("K", j), ("scores from the wrong tile", j, ring[st])
+            b, entries = j & 1, [k_index(j) + e for e in range(KE)]
+            for idx in entries:
+                yield from wait(("FULL", idx % NS), (idx // NS) & 1)
+            sts = [idx % NS for idx in entries]
+            for st in sts:
+                assert ring[st] == ("K", j), ("scores from the wrong tile", j, ring[st])
             for t in range(ntq):
                 if j >= 2:
                     name, parity = of_bar(t, j - 2)
                     yield from wait(name, parity)
                     assert pv_done.get(t, -1) >= j - 2, ("scores over probabilities still in use", t, j)
-                queues[2] += [("S", t, b, j, st), ("commit", ("SF", t, b)), ("commit", ("EMPTY", st))]
+                queues[2] += [("S", t, b, j, sts), ("commit", ("SF", t, b))] + [("commit", ("EMPTY", st)) for st in sts]
 
     def pv_issuer(t):
         for j in range(nsteps):
@@ -159,8 +161,8 @@ def simulate(nsteps, ntq, seed, product_barriers_per_tile=2, softmax_threads=2, 
             if op[0] == "commit":
                 bars[op[1]].arrive()
             elif op[0] == "S":
-                _, t, b, j, st = op
-                assert ring[st] == ("K", j), ("scores read a stage that was refilled", op, ring[st])
+                _, t, b, j, sts = op
+                assert all(ring[st] == ("K", j) for st in sts), ("scores read a stage that was refilled", op, ring)
                 scores[t, b] = j
             else:
                 _, t, b, j, st = op
@@ -189,6 +191,15 @@ def simulate(nsteps, ntq, seed, product_barriers_per_tile=2, softmax_threads=2, 
 def test_protocol_holds_under_random_schedules(nsteps, ntq):
     for seed in range(25):
         simulate(nsteps, ntq, seed)
+
+
+@pytest.mark.parametrize("stages,key_entries", [(4, 1), (5, 2)])
+@pytest.mark.parametrize("nsteps", [1, 2, 3, 5, 8, 21])
+def test_protocol_holds_with_short_rings(nsteps, stages, key_entries):
+    """Wide key rows leave room for four entries only, or for five of half a key tile."""
+    for ntq in (1, 2):
+        for seed in range(25):
+            simulate(nsteps, ntq, seed, NS=stages, KE=key_entries)
 
 
 def test_one_product_barrier_per_tile_is_not_enough():

@@ -72,6 +72,29 @@ __global__ void activation_rows_vec8_kernel(const __nv_bfloat16* __restrict__ in
 
 }  // namespace
 
+// out[i] = sum over s of part[s * stride + i], added in order
+template <typename T>
+__global__ void sum_partials_kernel(const float* __restrict__ part, int S, long long stride, T* __restrict__ out, long long n) {
+    TTIE_PDL_ENTRY();
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n) return;
+    float acc = 0.f;
+#pragma unroll 4
+    for (int s = 0; s < S; ++s) acc += part[s * stride + i];
+    out[i] = from_f32<T>(acc);
+}
+
+extern "C" int ttie_sum_partials(const float* part, int S, long long stride, void* out, long long n, int dtype, void* stream) {
+    if (n <= 0) return 0;
+    cudaStream_t s = (cudaStream_t)stream;
+    const unsigned blocks = (unsigned)((n + 127) / 128);
+    if (dtype == kF32) TTIE_LAUNCH(sum_partials_kernel<float>, blocks, 128, 0, s, part, S, stride, (float*)out, n);
+    else if (dtype == kBF16) TTIE_LAUNCH(sum_partials_kernel<__nv_bfloat16>, blocks, 128, 0, s, part, S, stride, (__nv_bfloat16*)out, n);
+    else TTIE_FAIL("sum_partials: unknown dtype %d", dtype);
+    TTIE_CHECK_LAUNCH("sum_partials");
+    return 0;
+}
+
 extern "C" int ttie_activation_rows(const void* in, long long ld, float* out, int T, int cols, int kind, float c, float scale, int dtype, void* stream) {
     if (T <= 0 || cols <= 0) return 0;
     if (kind < 0 || kind > 4) TTIE_FAIL("activation_rows: unknown kind %d", kind);

@@ -35,6 +35,9 @@ struct MmaParams {
     float* ws_o; float* ws_ml;
     int sigmoid;                        // 1 (tile loop only): a visible key weighs sigmoid(score + head_bias[head]), nothing is normalised
     const float* head_bias;             // [Hq] or null
+    int dv, per;                        // joint rows (dv > 0): of a row's output only the columns (h / per) * dv .. + dv of its head h are kept
+    __host__ __device__ __forceinline__ int out_width(int D) const { return dv > 0 ? dv : D; }
+    __device__ __forceinline__ int out_col0(int h) const { return dv > 0 ? h / per * dv : 0; }
 };
 
 __device__ __forceinline__ unsigned smem_addr(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
@@ -306,16 +309,19 @@ paged_attn_mma_kernel(const MmaParams p) {
         const int row = rrow[h];
         const int tok = row / G, g = row - tok * G;
         const size_t grow = (size_t)(q0 + tok) * p.Hq + kvh * G + g;
+        const int ow = p.out_width(D), oc = p.out_col0(kvh * G + g);
         if (p.num_splits == 1) {
             const float inv = p.sigmoid ? 1.f : l > 0.f ? 1.f / l : 0.f;
-            __nv_bfloat16* op = p.out + grow * D + 2 * (lane & 3);
+            __nv_bfloat16* op = p.out + grow * ow + 2 * (lane & 3) - oc;
 #pragma unroll
             for (int i = 0; i < D / 8; ++i)
-                *reinterpret_cast<__nv_bfloat162*>(op + i * 8) = __floats2bfloat162_rn(o[i][2 * h] * inv, o[i][2 * h + 1] * inv);
+                if (i * 8 >= oc && i * 8 < oc + ow)
+                    *reinterpret_cast<__nv_bfloat162*>(op + i * 8) = __floats2bfloat162_rn(o[i][2 * h] * inv, o[i][2 * h + 1] * inv);
         } else {
-            float* wo = p.ws_o + (grow * p.num_splits + split) * D + 2 * (lane & 3);
+            float* wo = p.ws_o + (grow * p.num_splits + split) * ow + 2 * (lane & 3) - oc;
 #pragma unroll
-            for (int i = 0; i < D / 8; ++i) *reinterpret_cast<float2*>(wo + i * 8) = make_float2(o[i][2 * h], o[i][2 * h + 1]);
+            for (int i = 0; i < D / 8; ++i)
+                if (i * 8 >= oc && i * 8 < oc + ow) *reinterpret_cast<float2*>(wo + i * 8) = make_float2(o[i][2 * h], o[i][2 * h + 1]);
             if ((lane & 3) == 0) {
                 float* ml = p.ws_ml + (grow * p.num_splits + split) * 2;
                 ml[0] = p.sigmoid ? 0.f : m_run[h] * 0.6931471805599453f;   // back to natural-log units for the merge
@@ -633,6 +639,8 @@ paged_attn_cluster_kernel(const MmaParams p) {
         const int r = (int)rank + lr * (int)C;
         const int row = row0 + r;
         if (row >= nrows) continue;
+        const int ow = p.out_width(D), oc = p.out_col0(kvh * G + row % G);
+        if (c4 * 4 < oc || c4 * 4 >= oc + ow) continue;
         float M = -INFINITY;
         for (unsigned k = 0; k < C; ++k) {
             const float2 ml = *reinterpret_cast<const float2*>(MLrecv + (k * rows_per_owner + lr) * 2);
@@ -650,7 +658,7 @@ paged_attn_cluster_kernel(const MmaParams p) {
         }
         const float inv = L > 0.f ? 1.f / L : 0.f;
         const int tok = row / G, g = row - tok * G;
-        __nv_bfloat16* dst = p.out + ((size_t)(q0 + tok) * p.Hq + kvh * G + g) * D + c4 * 4;
+        __nv_bfloat16* dst = p.out + ((size_t)(q0 + tok) * p.Hq + kvh * G + g) * ow + c4 * 4 - oc;
         uint2 w;
         w.x = pack_bf16(acc.x * inv, acc.y * inv);
         w.y = pack_bf16(acc.z * inv, acc.w * inv);
@@ -810,7 +818,7 @@ extern "C" int ttie_paged_attention_mma_weights(const void* q, long long q_strid
                                                 const int* block_table, int table_width, int page_size, const int* qsl,
                                                 const int* seq_lens, void* out, int T, int num_seqs, int Hq, int Hkv, int D,
                                                 int max_q_len, float scale, float softcap, int window, int chunk, int keep, int num_splits, int split_len,
-                                                float* scratch, int form, int weights, const float* head_bias, void* stream);
+                                                float* scratch, int form, int weights, const float* head_bias, int dv, int per, void* stream);
 
 extern "C" int ttie_paged_attention_mma_form(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
                                              const int* block_table, int table_width, int page_size, const int* qsl,
@@ -818,7 +826,7 @@ extern "C" int ttie_paged_attention_mma_form(const void* q, long long q_stride, 
                                              int max_q_len, float scale, float softcap, int window, int chunk, int num_splits, int split_len,
                                              float* scratch, int form, void* stream) {
     return ttie_paged_attention_mma_weights(q, q_stride, k_pages, v_pages, block_table, table_width, page_size, qsl, seq_lens, out, T, num_seqs,
-                                            Hq, Hkv, D, max_q_len, scale, softcap, window, chunk, 0, num_splits, split_len, scratch, form, 0, nullptr,
+                                            Hq, Hkv, D, max_q_len, scale, softcap, window, chunk, 0, num_splits, split_len, scratch, form, 0, nullptr, 0, 1,
                                             stream);
 }
 
@@ -826,7 +834,7 @@ extern "C" int ttie_paged_attention_mma_weights(const void* q, long long q_strid
                                                 const int* block_table, int table_width, int page_size, const int* qsl,
                                                 const int* seq_lens, void* out, int T, int num_seqs, int Hq, int Hkv, int D,
                                                 int max_q_len, float scale, float softcap, int window, int chunk, int keep, int num_splits, int split_len,
-                                                float* scratch, int form, int weights, const float* head_bias, void* stream) {
+                                                float* scratch, int form, int weights, const float* head_bias, int dv, int per, void* stream) {
     if (T <= 0 || num_seqs <= 0) return 0;
     if (weights != 0 && weights != 1) TTIE_FAIL("paged_attention_mma: unknown kind of weights %d", weights);
     if (weights == 1 && form != 0) TTIE_FAIL("paged_attention_mma: sigmoid weights run in the tile loop only");
@@ -848,7 +856,9 @@ extern "C" int ttie_paged_attention_mma_weights(const void* q, long long q_strid
     p.cap_in = softcap > 0.f ? scale / softcap : 0.f; p.cap_out = softcap > 0.f ? softcap / scale : 0.f;
     p.num_splits = num_splits; p.split_len = split_len;
     p.sigmoid = weights; p.head_bias = head_bias;
-    p.ws_o = scratch; p.ws_ml = scratch ? scratch + (size_t)T * Hq * num_splits * D : nullptr;
+    if (dv > 0 && (dv % 8 || per <= 0 || (long long)ceil_div(Hq, per) * dv > D)) TTIE_FAIL("paged_attention_mma: %d value columns per %d heads in rows of %d", dv, per, D);
+    p.dv = dv; p.per = per > 0 ? per : 1;
+    p.ws_o = scratch; p.ws_ml = scratch ? scratch + (size_t)T * Hq * num_splits * p.out_width(D) : nullptr;
     const int rows = max_q_len * (Hq / Hkv);
     if (form == 2 || form == 4) {
         if (num_splits > 1 && (split_len <= 0 || split_len % BN)) TTIE_FAIL("paged_attention_mma: the split length must be a multiple of %d", BN);
@@ -886,6 +896,6 @@ extern "C" int ttie_paged_attention_mma_weights(const void* q, long long q_strid
         default: TTIE_FAIL("paged_attention_mma: head size %d", D);
     }
     if (rc) return rc;
-    if (num_splits > 1) return attn_merge_bf16(p.ws_o, p.ws_ml, out, T * Hq, num_splits, D, s);
+    if (num_splits > 1) return attn_merge_bf16(p.ws_o, p.ws_ml, out, T * Hq, num_splits, dv > 0 ? dv : D, s);
     return 0;
 }

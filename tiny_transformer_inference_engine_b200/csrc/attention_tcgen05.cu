@@ -161,6 +161,13 @@ struct AttnTcParams {
     float* ws_o; float* ws_ml;                                   // partial results [row][split][D] and [row][split][2] (max in natural log, sum)
     int sigmoid;                                                 // 1: a visible key weighs sigmoid(score + head_bias[head]); no maximum, no rescaling, no division
     const float* head_bias;                                      // [Hq] or null
+    // Joint rows: keys and values of all kv heads side by side in one cache head.
+    int dv, per;                                                 // dv > 0: of a row's output only the columns (h / per) * dv .. + dv of its head h are kept
+    int joint;                                                   // 1 (two-tile kernel): row groups are the heads of one kv head; its values are columns kvh * DV ..
+    __host__ __device__ __forceinline__ int out_width(int D) const { return dv > 0 ? dv : D; }
+    __device__ __forceinline__ int out_col0(int h) const { return dv > 0 ? h / per * dv : 0; }
+    // first row of a page of this kv head in the page matrix, in pages' rows
+    __device__ __forceinline__ int page_row(int page, int kvh) const { return joint ? page * page_size : (page * Hkv + kvh) * page_size; }
 };
 
 // 1 / (1 + 2^-x): the sigmoid of a score in units of log2 e; x = -inf (a masked key) gives 1 / (1 + inf) = 0
@@ -190,7 +197,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
     // like none, and that wait ran out (seen once in several thousand launches of 600 CTAs).
     constexpr int KF = 0, KE = NST, VF = 2 * NST, VE = 3 * NST, SF = 4 * NST, SE = SF + 2, OF = SE + 2, OE = OF + 2, PF = OE + 2,
                   XB = PF + 2, XL = XB + 2, NBARS = XL + 1;
-    constexpr int CB = D / 64;                                   // 64-column blocks of the head dimension
+    constexpr int CB = D / 64, DO = D;                           // 64-column blocks of the head dimension; output columns
     constexpr uint32_t KVBLK = BN * 128;                         // bytes of one 64-column block of a key / value tile
     constexpr uint32_t KV_BYTES = CB * KVBLK;
     const uint32_t QBLK = (uint32_t)p.q_rows * 128;              // ... of the staged query rows
@@ -227,12 +234,13 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
         // (only with splits) no key of this split is visible: an empty partial result, nothing allocated.  The scratch
         // memory may still be read by the merge kernel of the launch before this one: wait for it first.
         pdl_wait();
-        for (int e = threadIdx.x; e < rows_here * D; e += blockDim.x) {
-            const int r = e / D, row = row0 + r;
+        const int ow = p.out_width(DO);
+        for (int e = threadIdx.x; e < rows_here * ow; e += blockDim.x) {
+            const int r = e / ow, row = row0 + r;
             const int tok = row / G, g = row - tok * G;
             const size_t grow = (size_t)(q0 + tok) * p.Hq + kvh * G + g;
-            p.ws_o[(grow * p.num_splits + split) * D + (e - r * D)] = 0.f;
-            if (e - r * D == 0) {                                  // (sigmoid weights: an empty piece still counts as one of the pieces that add)
+            p.ws_o[(grow * p.num_splits + split) * ow + (e - r * ow)] = 0.f;
+            if (e - r * ow == 0) {                                 // (sigmoid weights: an empty piece still counts as one of the pieces that add)
                 p.ws_ml[(grow * p.num_splits + split) * 2] = p.sigmoid ? 0.f : -INFINITY;
                 p.ws_ml[(grow * p.num_splits + split) * 2 + 1] = p.sigmoid ? 1.0f / (float)p.num_splits : 0.f;
             }
@@ -269,7 +277,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
                 const int key = span.key(v_lo + jt * BN) + bx * box_rows;
                 const int pg = key / ps;
                 const int page = pg < p.table_width ? p.block_table[(size_t)seq * p.table_width + pg] : 0;
-                y_first = (page * p.Hkv + kvh) * ps + (key - pg * ps);
+                y_first = p.page_row(page, kvh) + (key - pg * ps);
             }
         }
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_slot)), "r"(TMEM_COLS) : "memory");
@@ -313,7 +321,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
                 const int key = span.key(v_lo + j * BN) + lane * box_rows;
                 const int pg = key / ps;
                 const int page = pg < p.table_width ? table[pg] : 0;
-                y = (page * p.Hkv + kvh) * ps + (key - pg * ps);
+                y = p.page_row(page, kvh) + (key - pg * ps);
             }
             return y;
         };
@@ -357,7 +365,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
                 const int key = span.key(v_lo + j * BN) + lane * box_rows;
                 const int pg = key / ps;
                 const int page = pg < p.table_width ? table[pg] : 0;
-                y = (page * p.Hkv + kvh) * ps + (key - pg * ps);
+                y = p.page_row(page, kvh) + (key - pg * ps);
             }
             return y;
         };
@@ -579,9 +587,12 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
         }
         if (ok && valid && p.num_splits > 1) {
             const size_t grow = (size_t)(q0 + tok) * p.Hq + kvh * G + g;
-            float* dst = p.ws_o + (grow * p.num_splits + split) * D + part * OC;
+            const int ow = p.out_width(D), oc = part * OC - p.out_col0(kvh * G + g);
+            if (oc >= 0 && oc < ow) {
+                float* dst = p.ws_o + (grow * p.num_splits + split) * ow + oc;
 #pragma unroll
-            for (int i = 0; i < OC; i += 4) *reinterpret_cast<float4*>(dst + i) = make_float4(o[i], o[i + 1], o[i + 2], o[i + 3]);
+                for (int i = 0; i < OC; i += 4) *reinterpret_cast<float4*>(dst + i) = make_float4(o[i], o[i + 1], o[i + 2], o[i + 3]);
+            }
             if (part == 0) {
                 float* ml = p.ws_ml + (grow * p.num_splits + split) * 2;
                 ml[0] = m_run * 0.6931471805599453f;                 // natural-log units for the merge
@@ -589,7 +600,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
             }
         } else if (ok && valid) {
             const float inv = l_tot > 0.f ? 1.f / l_tot : 0.f;
-            __nv_bfloat16* dst = p.out + ((size_t)(q0 + tok) * p.Hq + kvh * G + g) * D + part * OC;
+            const int ow = p.out_width(D), oc = part * OC - p.out_col0(kvh * G + g);
+            __nv_bfloat16* dst = p.out + ((size_t)(q0 + tok) * p.Hq + kvh * G + g) * ow + oc;
+            if (oc >= 0 && oc < ow)
 #pragma unroll
             for (int i = 0; i < OC; i += 8) {
                 uint32_t w[4];
@@ -638,6 +651,13 @@ constexpr int NS = 8;                                            // stages of th
 enum { PP_FULL = 0, PP_EMPTY = NS, PP_SF = 2 * NS, PP_PF = PP_SF + 4, PP_SC = PP_PF + 4, PP_OC = PP_SC + 4, PP_OF = PP_OC + 4,
        PP_LF = PP_OF + 4, PP_NBARS = PP_LF + 2 };                // SF, PF, SC, OC, OF: [tile][step parity]
 constexpr int PP_NTHREADS = 512;
+// What 227 KB leave beside NT query tiles: with two tiles of 256-column rows a key tile travels as two entries of the ring (128
+// columns each), so that five entries of 16 KB fit.
+__host__ __device__ constexpr int key_entries(int D, int NT) { return D > 128 && NT > 1 ? 2 : 1; }
+__host__ __device__ constexpr int ring_stages(int D, int NT) { return D > 128 ? (NT > 1 ? 5 : 4) : NS; }
+__host__ __device__ constexpr int entry_blocks(int D, int DO, int NT) {          // 64-column blocks of an entry
+    return D / 64 / key_entries(D, NT) > DO / 64 ? D / 64 / key_entries(D, NT) : DO / 64;
+}
 constexpr float RESCALE_LOG2 = 8.f;                              // a row's output is rescaled when its maximum grew by more
 }
 
@@ -661,19 +681,20 @@ __device__ __forceinline__ void tmem_st32(uint32_t taddr, const uint32_t (&r)[32
                    "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31]) : "memory");
 }
 
-// NT: query tiles per CTA.  Tensor memory holds 2 x 2 x 64 score columns and NT x D output columns: two tiles up to
-// head size 128, one tile (its scores at columns 0..127, its output at 256..511) at head size 256.
-template <int D, int NT>
+// D: key size; DO: value columns (D, or fewer: the value columns of one kv head of a joint row).  NT: query tiles per CTA.  Tensor
+// memory holds 2 x 2 x 64 score columns and NT x DO output columns: two tiles up to 128 output columns, one tile (its scores
+// at columns 0..127, its output at 256..511) at 256.
+template <int D, int DO, int NT>
 __global__ void __launch_bounds__(pp::PP_NTHREADS, 1)
 attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const AttnTcParams p) {
     using namespace pp;
-    static_assert(256 + NT * D <= 512, "tensor memory: scores of two tiles, then the output tiles");
-    constexpr int NSD = D > 128 ? 4 : NS;                        // ring stages in use (a stage is D x 64 x 2 bytes)
-    constexpr int CB = D / 64;
+    static_assert(256 + NT * DO <= 512, "tensor memory: scores of two tiles, then the output tiles");
+    constexpr int NSD = ring_stages(D, NT), KE = key_entries(D, NT);      // ring entries in use; entries of a key tile
+    constexpr int CB = D / 64, CBK = CB / KE, CBV = DO / 64;     // 64-column blocks of a row, of a key entry, of a value tile
     constexpr uint32_t QBLK = BM * 128, KVBLK = BNK * 128;       // bytes of one 64-column block of a query / key tile
-    constexpr uint32_t QT_BYTES = CB * QBLK, KV_BYTES = CB * KVBLK;
+    constexpr uint32_t QT_BYTES = CB * QBLK, KV_BYTES = entry_blocks(D, DO, NT) * KVBLK, K_BYTES = CBK * KVBLK, V_BYTES = CBV * KVBLK;
     constexpr uint32_t TMEM_COLS = 512;
-    constexpr uint32_t S_COL = 0, O_COL = 256;                   // scores of (tile t, buffer b) at t * 128 + b * 64; output of tile t at 256 + t * D
+    constexpr uint32_t S_COL = 0, O_COL = 256;                   // scores of (tile t, buffer b) at t * 128 + b * 64; output of tile t at 256 + t * DO
     extern __shared__ unsigned char smem_dyn[];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_dyn) + 1023) & ~(uintptr_t)1023);
     unsigned char* Qs = smem;                                    // [NT tiles]
@@ -704,12 +725,13 @@ attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
         // (only with splits) no key of this split is visible: an empty partial result, nothing allocated.  The scratch
         // memory may still be read by the merge kernel of the launch before this one: wait for it first.
         pdl_wait();
-        for (int e = threadIdx.x; e < rows_here * D; e += blockDim.x) {
-            const int r = e / D, row = row0 + r;
+        const int ow = p.out_width(DO);
+        for (int e = threadIdx.x; e < rows_here * ow; e += blockDim.x) {
+            const int r = e / ow, row = row0 + r;
             const int tok = row / G, g = row - tok * G;
             const size_t grow = (size_t)(q0 + tok) * p.Hq + kvh * G + g;
-            p.ws_o[(grow * p.num_splits + split) * D + (e - r * D)] = 0.f;
-            if (e - r * D == 0) {                                  // (sigmoid weights: an empty piece still counts as one of the pieces that add)
+            p.ws_o[(grow * p.num_splits + split) * ow + (e - r * ow)] = 0.f;
+            if (e - r * ow == 0) {                                 // (sigmoid weights: an empty piece still counts as one of the pieces that add)
                 p.ws_ml[(grow * p.num_splits + split) * 2] = p.sigmoid ? 0.f : -INFINITY;
                 p.ws_ml[(grow * p.num_splits + split) * 2 + 1] = p.sigmoid ? 1.0f / (float)p.num_splits : 0.f;
             }
@@ -871,13 +893,13 @@ attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
                     if (!ok) break;
                     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
-                    for (int c = 0; c < D / 32; ++c) {
+                    for (int c = 0; c < DO / 32; ++c) {
                         uint32_t ov[32];
-                        tmem_ld32(lane_addr + O_COL + t * D + c * 32, ov);
+                        tmem_ld32(lane_addr + O_COL + t * DO + c * 32, ov);
                         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
                         for (int i = 0; i < 32; ++i) ov[i] = __float_as_uint(__uint_as_float(ov[i]) * a);
-                        tmem_st32(lane_addr + O_COL + t * D + c * 32, ov);
+                        tmem_st32(lane_addr + O_COL + t * DO + c * 32, ov);
                     }
                     asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
                 }
@@ -898,20 +920,21 @@ attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
             const float l_tot = lsum_s[t][r];
             const bool partial = p.num_splits > 1;
             const float inv = partial ? 1.f : (l_tot > 0.f ? 1.f / l_tot : 0.f);
+            const int ow = p.out_width(DO), oc = valid ? p.out_col0(kvh * G + g) : 0;
 #pragma unroll
-            for (int c = 0; c < D / 32; ++c) {
+            for (int c = 0; c < DO / 32; ++c) {
                 uint32_t ov[32];
-                tmem_ld32(lane_addr + O_COL + t * D + c * 32, ov);
+                tmem_ld32(lane_addr + O_COL + t * DO + c * 32, ov);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-                if (!valid) continue;
+                if (!valid || c * 32 < oc || c * 32 >= oc + ow) continue;
                 if (partial) {
-                    float* dst = p.ws_o + (grow * p.num_splits + split) * D + c * 32;
+                    float* dst = p.ws_o + (grow * p.num_splits + split) * ow + c * 32 - oc;
 #pragma unroll
                     for (int i = 0; i < 32; i += 4)
                         *reinterpret_cast<float4*>(dst + i) = make_float4(__uint_as_float(ov[i]), __uint_as_float(ov[i + 1]),
                                                                           __uint_as_float(ov[i + 2]), __uint_as_float(ov[i + 3]));
                 } else {
-                    __nv_bfloat16* dst = p.out + grow * D + c * 32;
+                    __nv_bfloat16* dst = p.out + grow * ow + c * 32 - oc;
 #pragma unroll
                     for (int i = 0; i < 32; i += 8) {
                         uint32_t w[4];
@@ -945,33 +968,41 @@ attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
                     const int key = span.key(v_lo + j * BNK) + lane * box_rows;
                     const int pg = key / ps;
                     const int page = pg < p.table_width ? table[pg] : 0;
-                    y = (page * p.Hkv + kvh) * ps + (key - pg * ps);
+                    y = p.page_row(page, kvh) + (key - pg * ps);
                 }
                 return y;
             };
             int it = 0;                                         // tiles copied so far
-            auto emit = [&](const CUtensorMap* map, int y_lane, int code) -> bool {
+            const int v_x = p.joint ? kvh * DO : 0;             // first value column
+            auto emit_entry = [&](const CUtensorMap* map, int y_lane, int code, bool values, int part) -> bool {
                 const int st = it % NSD;
                 int ok = 1;
                 if (lane == 0) ok = mbar_wait_relaxed(BAR(PP_EMPTY + st), ((it / NSD) & 1) ^ 1, code);
                 if (!__shfl_sync(0xffffffffu, ok, 0)) return false;
-                if (lane == 0) mbar_expect_tx(BAR(PP_FULL + st), KV_BYTES);
+                if (lane == 0) mbar_expect_tx(BAR(PP_FULL + st), values ? V_BYTES : K_BYTES);
                 __syncwarp();
                 if (lane < nboxes) {                                // every lane issues the copies of its own box
 #pragma unroll
-                    for (int cb = 0; cb < CB; ++cb)
-                        tma_load_2d(smem_u32(ring + st * KV_BYTES + cb * KVBLK + lane * box_rows * 128), map, BAR(PP_FULL + st), cb * 64, y_lane);
+                    for (int cb = 0; cb < entry_blocks(D, DO, NT); ++cb)
+                        if (cb < (values ? CBV : CBK))
+                            tma_load_2d(smem_u32(ring + st * KV_BYTES + cb * KVBLK + lane * box_rows * 128), map, BAR(PP_FULL + st),
+                                        (values ? v_x : part * CBK * 64) + cb * 64, y_lane);
                 }
                 ++it;
                 return true;
             };
+            auto emit = [&](const CUtensorMap* map, int y_lane, int code, bool values) -> bool {
+                bool ok = true;
+                for (int part = 0; part < (values ? 1 : KE) && ok; ++part) ok = emit_entry(map, y_lane, code, values, part);
+                return ok;
+            };
             int y0 = box_row(0), y1 = box_row(1), y2 = box_row(2);   // tiles j, j+1, j+2
-            bool go = emit(&tmK, y0, 1);
-            if (go && nsteps > 1) go = emit(&tmK, y1, 1);
+            bool go = emit(&tmK, y0, 1, false);
+            if (go && nsteps > 1) go = emit(&tmK, y1, 1, false);
             for (int j = 0; j < nsteps && go; ++j) {
                 const int y3 = box_row(j + 3);
-                go = emit(&tmV, y0, 2);
-                if (go && j + 2 < nsteps) go = emit(&tmK, y2, 1);
+                go = emit(&tmV, y0, 2, true);
+                if (go && j + 2 < nsteps) go = emit(&tmK, y2, 1, false);
                 y0 = y1; y1 = y2; y2 = y3;
             }
         } else if (lane == 0) {
@@ -986,10 +1017,10 @@ attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
             // A product of 48-64 clocks leaves its thread a dozen instructions: the descriptors' upper words are
             // constants, the lower words are one addition away from values kept in registers.
             constexpr uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(BNK >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
-            constexpr uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(D >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
-            // position of a tile in the ring's order K0 K1 V0 K2 V1 K3 ... V(n-2) V(n-1)
-            auto k_index = [&](int j) { return j < 2 ? j : 2 * j - 1; };
-            auto v_index = [&](int j) { return j == nsteps - 1 ? 2 * nsteps - 1 : 2 * j + 2; };
+            constexpr uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(DO >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
+            // position of a tile (its first entry) in the ring's order K0 K1 V0 K2 V1 K3 ... V(n-2) V(n-1)
+            auto k_index = [&](int j) { return j < 2 ? KE * j : KE * 2 + (KE + 1) * (j - 2) + 1; };
+            auto v_index = [&](int j) { return j == nsteps - 1 ? (KE + 1) * nsteps - 1 : KE * 2 + (KE + 1) * j; };
             if (warp == 15) {
                 uint32_t q_lo[NT][CB];                          // lower descriptor words of the query blocks
 #pragma unroll
@@ -998,10 +1029,18 @@ attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
                     for (int cb = 0; cb < CB; ++cb) q_lo[t][cb] = desc_lo(smem_u32(Qs + t * QT_BYTES + cb * QBLK), 16);
                 const uint32_t ring_k_lo = desc_lo(smem_u32(ring), 16);
                 for (int j = 0; j < nsteps; ++j) {
-                    const int b = j & 1, idx = k_index(j), st = idx % NSD;
-                    if (!mbar_wait(BAR(PP_FULL + st), (idx / NSD) & 1, 3)) break;
-                    const uint32_t k_lo = ring_k_lo + (uint32_t)st * (KV_BYTES >> 4);
+                    const int b = j & 1;
+                    int st[KE];
+                    uint32_t k_lo[KE];
                     bool ok = true;
+#pragma unroll
+                    for (int e = 0; e < KE; ++e) {
+                        const int idx = k_index(j) + e;
+                        st[e] = idx % NSD;
+                        k_lo[e] = ring_k_lo + (uint32_t)st[e] * (KV_BYTES >> 4);
+                        ok = ok && mbar_wait(BAR(PP_FULL + st[e]), (idx / NSD) & 1, 3);
+                    }
+                    if (!ok) break;
 #pragma unroll
                     for (int t = 0; t < NT; ++t) {
                         if (t < ntq) {
@@ -1013,11 +1052,13 @@ attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
                             for (int cb = 0; cb < CB; ++cb)
 #pragma unroll
                                 for (int k = 0; k < 4; ++k) {
-                                    if (cb | k) umma_ss_lean<true>(d, q_lo[t][cb] + 2 * k, k_lo + cb * (KVBLK >> 4) + 2 * k, idesc_s);
-                                    else umma_ss_lean<false>(d, q_lo[t][cb] + 2 * k, k_lo + cb * (KVBLK >> 4) + 2 * k, idesc_s);
+                                    const uint32_t kb = k_lo[cb / CBK] + (cb % CBK) * (KVBLK >> 4) + 2 * k;
+                                    if (cb | k) umma_ss_lean<true>(d, q_lo[t][cb] + 2 * k, kb, idesc_s);
+                                    else umma_ss_lean<false>(d, q_lo[t][cb] + 2 * k, kb, idesc_s);
                                 }
                             umma_commit(BAR(PP_SF + 2 * t + b));
-                            umma_commit(BAR(PP_EMPTY + st));           // one arrival per tile in use
+#pragma unroll
+                            for (int e = 0; e < KE; ++e) umma_commit(BAR(PP_EMPTY + st[e]));           // one arrival per tile in use
                         }
                     }
                     if (!ok) break;
@@ -1025,7 +1066,7 @@ attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
             } else if (warp - 13 < ntq) {
                 const int t = warp - 13;
                 const uint32_t ring_v_lo = desc_lo(smem_u32(ring), KVBLK);
-                const uint32_t s_tmem = tmem_base + S_COL + (uint32_t)t * 128, o_tmem = tmem_base + O_COL + (uint32_t)t * D;
+                const uint32_t s_tmem = tmem_base + S_COL + (uint32_t)t * 128, o_tmem = tmem_base + O_COL + (uint32_t)t * DO;
                 for (int j = 0; j < nsteps; ++j) {
                     const int b = j & 1, idx = v_index(j), st = idx % NSD;
                     const uint32_t par = (j >> 1) & 1;
@@ -1118,11 +1159,11 @@ int launch(const CUtensorMap& mk, const CUtensorMap& mv, const AttnTcParams& p, 
     TTIE_CHECK_LAUNCH("attention_tc");
     return 0;
 }
-template <int D>
+template <int D, int DO>
 int launch_pp(const CUtensorMap& mk, const CUtensorMap& mv, const AttnTcParams& p, cudaStream_t s) {
-    constexpr int NT = D > 128 ? 1 : 2, NSD = D > 128 ? 4 : pp::NS;
-    const size_t smem = NT * (size_t)(D / 64) * BM * 128 + NSD * (size_t)(D / 64) * pp::BNK * 128 + 1024;
-    auto k = attn_tc_pp_kernel<D, NT>;
+    constexpr int NT = DO > 128 ? 1 : 2, NSD = pp::ring_stages(D, NT);
+    const size_t smem = NT * (size_t)(D / 64) * BM * 128 + NSD * (size_t)pp::entry_blocks(D, DO, NT) * pp::BNK * 128 + 1024;
+    auto k = attn_tc_pp_kernel<D, DO, NT>;
     static bool allowed[64] = {false};                           // the attribute is set once per device
     int dev = 0;
     if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) dev = 0;
@@ -1182,11 +1223,14 @@ extern "C" int ttie_attn_tc_supported(int D, int page_size) {
 // num_splits > 1: the key range is cut into pieces of split_len keys (a multiple of 128) over grid y; the partial
 // results go to `scratch` (ttie_attn_scratch_floats) and a merge kernel writes `out`.
 // weights 0: softmax; 1: sigmoid(score + head_bias[head]) per visible key (head_bias float32 [Hq] or null)
+// Joint rows (one cache head holds the rows of all kv heads side by side; D is that row's width).  dv > 0 (a multiple of 32): with
+// Hkv 1, head h's output is the columns (h / per) * dv .. of its row only; out is [T, Hq, dv].  joint = 64 or 128 (two_tiles only):
+// Hkv row groups, one per kv head, whose values are the columns kvh * joint .. + joint; out is [T, Hq, joint].
 extern "C" int ttie_paged_attention_tc_weights(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
                                                int num_pages, const int* block_table, int table_width, int page_size, const int* qsl,
                                                const int* seq_lens, void* out, int T, int num_seqs, int Hq, int Hkv, int D,
                                                int max_q_len, float scale, float softcap, int window, int chunk, int keep, int num_splits, int split_len,
-                                               float* scratch, int two_tiles, int weights, const float* head_bias, void* stream);
+                                               float* scratch, int two_tiles, int weights, const float* head_bias, int dv, int per, int joint, void* stream);
 
 extern "C" int ttie_paged_attention_tc(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
                                        int num_pages, const int* block_table, int table_width, int page_size, const int* qsl,
@@ -1195,14 +1239,14 @@ extern "C" int ttie_paged_attention_tc(const void* q, long long q_stride, const 
                                        int two_tiles, void* stream) {
     return ttie_paged_attention_tc_weights(q, q_stride, k_pages, v_pages, num_pages, block_table, table_width, page_size, qsl, seq_lens, out, T,
                                            num_seqs, Hq, Hkv, D, max_q_len, scale, softcap, window, chunk, 0, num_splits, split_len, scratch,
-                                           two_tiles, 0, nullptr, stream);
+                                           two_tiles, 0, nullptr, 0, 1, 0, stream);
 }
 
 extern "C" int ttie_paged_attention_tc_weights(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
                                                int num_pages, const int* block_table, int table_width, int page_size, const int* qsl,
                                                const int* seq_lens, void* out, int T, int num_seqs, int Hq, int Hkv, int D,
                                                int max_q_len, float scale, float softcap, int window, int chunk, int keep, int num_splits, int split_len,
-                                               float* scratch, int two_tiles, int weights, const float* head_bias, void* stream) {
+                                               float* scratch, int two_tiles, int weights, const float* head_bias, int dv, int per, int joint, void* stream) {
     if (T <= 0 || num_seqs <= 0) return 0;
     if (weights != 0 && weights != 1) TTIE_FAIL("attention_tc: unknown kind of weights %d", weights);
     if (!ttie_attn_tc_supported(D, page_size)) TTIE_FAIL("attention_tc: head size %d with pages of %d keys is not supported", D, page_size);
@@ -1215,7 +1259,10 @@ extern "C" int ttie_paged_attention_tc_weights(const void* q, long long q_stride
         TTIE_FAIL("attention_tc: splits need scratch and a split length that is a multiple of %d", BN);
     if (num_splits > 65535) TTIE_FAIL("attention_tc: too many splits (%d)", num_splits);
     CUtensorMap mk, mv;
-    const long long rows = (long long)num_pages * Hkv * page_size;
+    if (dv > 0 && (dv % 32 || per <= 0 || (long long)ceil_div(Hq, per) * dv > D)) TTIE_FAIL("attention_tc: %d value columns per %d heads in rows of %d", dv, per, D);
+    if (joint && (!two_tiles || (joint != 64 && joint != 128) || (D != 128 && D != 256) || (long long)Hkv * joint > D))
+        TTIE_FAIL("attention_tc: %d kv heads of %d value columns in joint rows of %d are not supported", Hkv, joint, D);
+    const long long rows = (long long)num_pages * (joint ? 1 : Hkv) * page_size;
     const int tile_keys = two_tiles ? pp::BNK : BN;              // keys per copy tile of the kernel
     const int box_rows = page_size < tile_keys ? page_size : tile_keys;
     if (make_page_map(&mk, k_pages, rows, D, box_rows)) return -1;
@@ -1226,20 +1273,24 @@ extern "C" int ttie_paged_attention_tc_weights(const void* q, long long q_stride
     p.num_seqs = num_seqs; p.Hq = Hq; p.Hkv = Hkv; p.scale_log2 = scale * 1.4426950408889634f; p.window = window; p.chunk = chunk;
     p.keep = window > 0 ? keep : 0;
     p.cap_in = softcap > 0.f ? scale / softcap : 0.f; p.cap_out = softcap > 0.f ? softcap / scale : 0.f;
-    p.row_tiles = ceil_div(max_q_len * (Hq / Hkv), two_tiles && D <= 128 ? 2 * BM : BM);
+    p.row_tiles = ceil_div(max_q_len * (Hq / Hkv), two_tiles && (D <= 128 || joint) ? 2 * BM : BM);
     p.num_splits = num_splits; p.split_len = split_len;
     p.sigmoid = weights; p.head_bias = head_bias;
-    p.ws_o = scratch; p.ws_ml = scratch ? scratch + (size_t)T * Hq * num_splits * D : nullptr;
+    p.dv = dv; p.per = per > 0 ? per : 1; p.joint = joint ? 1 : 0;
+    const int out_width = joint ? joint : p.out_width(D);
+    p.ws_o = scratch; p.ws_ml = scratch ? scratch + (size_t)T * Hq * num_splits * out_width : nullptr;
     if ((long long)num_seqs * Hkv * p.row_tiles > 2147483647LL) TTIE_FAIL("attention_tc: grid too large");
     cudaStream_t s = (cudaStream_t)stream;
     const int rows_most = max_q_len * (Hq / Hkv);
     const bool ahead = rows_most >= BM;                          // full row tiles: a prompt portion
     p.q_rows = ahead ? BM : 32 * ceil_div(rows_most, 32);
-    const int rc = two_tiles ? (D == 64 ? launch_pp<64>(mk, mv, p, s) : D == 128 ? launch_pp<128>(mk, mv, p, s) : launch_pp<256>(mk, mv, p, s))
+    const int rc = joint ? (D == 256 ? (joint == 128 ? launch_pp<256, 128>(mk, mv, p, s) : launch_pp<256, 64>(mk, mv, p, s))
+                                     : (joint == 128 ? launch_pp<128, 128>(mk, mv, p, s) : launch_pp<128, 64>(mk, mv, p, s)))
+                 : two_tiles ? (D == 64 ? launch_pp<64, 64>(mk, mv, p, s) : D == 128 ? launch_pp<128, 128>(mk, mv, p, s) : launch_pp<256, 256>(mk, mv, p, s))
                  : D == 64 ? (ahead ? launch<64, true, 2>(mk, mv, p, s) : launch<64, false, 4>(mk, mv, p, s))
                            : (ahead ? launch<128, true, 2>(mk, mv, p, s)
                                     : p.q_rows <= 64 ? launch<128, false, 3>(mk, mv, p, s) : launch<128, false, 2>(mk, mv, p, s));
     if (rc) return rc;
-    if (num_splits > 1) return attn_merge_bf16(p.ws_o, p.ws_ml, out, T * Hq, num_splits, D, s);
+    if (num_splits > 1) return attn_merge_bf16(p.ws_o, p.ws_ml, out, T * Hq, num_splits, out_width, s);
     return 0;
 }

@@ -814,6 +814,44 @@ __global__ void __launch_bounds__(256) row_norm_gate_kernel(const float* __restr
     }
 }
 
+// ... with eight values per thread (bfloat16 gate; n a multiple of 8, 16-byte aligned rows): one trip to memory per row
+__global__ void __launch_bounds__(1024) row_norm_gate_vec8_kernel(const float* __restrict__ o, const __nv_bfloat16* __restrict__ gate, long long ld_g,
+                                                                  const float* __restrict__ w, int n, float eps, int act, __nv_bfloat16* __restrict__ out) {
+    __shared__ float scratch[32];
+    const int j = threadIdx.x * 8;
+    const bool in = j < n;
+    float wv[8];
+#pragma unroll
+    for (int i = 0; i < 8; i += 4) {                                 // (weights do not depend on the kernel before this one)
+        const float4 x = (w && in) ? *reinterpret_cast<const float4*>(w + j + i) : make_float4(1.f, 1.f, 1.f, 1.f);
+        wv[i] = x.x; wv[i + 1] = x.y; wv[i + 2] = x.z; wv[i + 3] = x.w;
+    }
+    TTIE_PDL_ENTRY();
+    const float* src = o + (size_t)blockIdx.x * n + j;
+    float v[8], ss = 0.f;
+    uint4 graw = make_uint4(0u, 0u, 0u, 0u);
+    if (in) graw = *reinterpret_cast<const uint4*>(gate + (size_t)blockIdx.x * ld_g + j);
+#pragma unroll
+    for (int i = 0; i < 8; i += 4) {
+        const float4 x = in ? *reinterpret_cast<const float4*>(src + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        v[i] = x.x; v[i + 1] = x.y; v[i + 2] = x.z; v[i + 3] = x.w;
+        ss += (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
+    }
+    ss = block_sum(ss, scratch);
+    if (!in) return;
+    const float inv = 1.0f / sqrtf(ss / (float)n + eps);
+    const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&graw);
+    uint4 packed;
+    __nv_bfloat162* y2 = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        const float2 g = __bfloat1622float2(g2[k]);
+        const float s0 = 1.0f / (1.0f + expf(-g.x)), s1 = 1.0f / (1.0f + expf(-g.y));
+        y2[k] = __floats2bfloat162_rn(v[2 * k] * inv * wv[2 * k] * (act == 0 ? g.x * s0 : s0), v[2 * k + 1] * inv * wv[2 * k + 1] * (act == 0 ? g.y * s1 : s1));
+    }
+    *reinterpret_cast<uint4*>(out + (size_t)blockIdx.x * n + j) = packed;
+}
+
 // Key channels per thread for heads of D key channels: the fewest (the most threads per state) whose slices still fit a warp.
 int keys_per_thread(int D) { return D <= 128 ? 4 : D <= 256 ? 8 : 16; }
 
@@ -1004,6 +1042,11 @@ extern "C" int ttie_head_norm_gate(const float* o, const void* gate, long long l
     cudaStream_t s = (cudaStream_t)stream;
     if (H == 1 && Dv > 256 && Dv <= 8192) {
         if (dtype != kF32 && dtype != kBF16) TTIE_FAIL("head_norm_gate: unknown dtype %d", dtype);
+        if (dtype == kBF16 && Dv % 8 == 0 && ld_g % 8 == 0 && !(((uintptr_t)o | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)out) & 15)) {
+            TTIE_LAUNCH(row_norm_gate_vec8_kernel, T, (Dv / 8 + 31) / 32 * 32, 0, s, o, (const __nv_bfloat16*)gate, ld_g, w, Dv, eps, act, (__nv_bfloat16*)out);
+            TTIE_CHECK_LAUNCH("head_norm_gate");
+            return 0;
+        }
 #define RNG(TT, PER) TTIE_LAUNCH((row_norm_gate_kernel<TT, PER>), T, 256, 0, s, o, (const TT*)gate, ld_g, w, Dv, eps, act, (TT*)out)
         if (Dv <= 1024) { if (dtype == kF32) RNG(float, 4); else RNG(__nv_bfloat16, 4); }
         else if (Dv <= 4096) { if (dtype == kF32) RNG(float, 16); else RNG(__nv_bfloat16, 16); }

@@ -56,13 +56,13 @@ _SIGNATURES = {
                                      _c_void, _c_int, _c_int, _c_void, _c_void],
     "ttie_paged_attention_mma_weights": [_c_void, _c_ll, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_void, _c_void,
                                          _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_int, _c_int, _c_int, _c_int,
-                                         _c_void, _c_int, _c_int, _c_void, _c_void],
+                                         _c_void, _c_int, _c_int, _c_void, _c_int, _c_int, _c_void],
     "ttie_paged_attention_tc": [_c_void, _c_ll, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_void, _c_void, _c_void,
                                 _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int,
                                 _c_void],
     "ttie_paged_attention_tc_weights": [_c_void, _c_ll, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_void, _c_void, _c_void,
                                         _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int,
-                                        _c_int, _c_void, _c_void],
+                                        _c_int, _c_void, _c_int, _c_int, _c_int, _c_void],
     "ttie_gemm_tc": [_c_void, _c_ll, _c_void, _c_ll, _c_void, _c_void, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void],
     "ttie_gemm_tc_pair": [_c_void, _c_ll, _c_void, _c_ll, _c_void, _c_void, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void],
     "ttie_scale_add_layernorm": [_c_void, _c_void, _c_int, _c_void, _c_int, _c_ll, _c_void, _c_void, _c_void, _c_int, _c_void, _c_int,
@@ -90,6 +90,7 @@ _SIGNATURES = {
     "ttie_attn_joint_tile_rows": [_c_int, _c_int],
     "ttie_paged_attention_joint": [_c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int,
                                    _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int, _c_void],
+    "ttie_sum_partials": [_c_void, _c_int, _c_ll, _c_void, _c_ll, _c_int, _c_void],
     "ttie_activation_rows": [_c_void, _c_ll, _c_void, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_void],
     "ttie_rglru_scan": [_c_void, _c_void, _c_void, _c_void, _c_int, _c_void, _c_void, _c_ll, _c_int, _c_void, _c_ll, _c_int, _c_void,
                         _c_int, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void, _c_int, _c_void,
@@ -435,6 +436,17 @@ class CudaOps:
         if bias is not None:
             return torch.addmm(bias, x, w.t())
         return torch.mm(x, w.t())
+
+    def linear_narrow(self, x, w):
+        """x @ w.T for a matrix of few rows and many columns, in the compute dtype: for few rows of x the K range is cut over CTAs (a
+        few hundred matrix rows alone leave most of the GPU idle) and one small kernel adds the pieces."""
+        y = self.linear(x, w, None, partial_ok=True)
+        if y.dim() == 2:
+            return y
+        out = torch.empty(y.shape[1:], dtype=x.dtype, device=x.device)
+        self._check(self.lib.ttie_sum_partials(_ptr(y), y.shape[0], y.stride(0), _ptr(out), out.numel(), self._dt(out), self._stream(x)), "sum_partials")
+        self.launches += 1
+        return out
 
     def linear_tc(self, x, w, bias, out_dtype=None, tile_n=256):
         """The tcgen05 / TMA / TMEM product: y = x @ w.T (+ bias) for bfloat16 operands."""
@@ -845,13 +857,15 @@ class CudaOps:
 
     def paged_attention(self, qkv, num_heads, num_kv_heads, head_dim, k_pages, v_pages, block_table, page_size,
                         query_start_loc, seq_lens, num_seqs, max_q_len, max_kv_len, scale, window, out,
-                        plan=None, softcap=0.0, chunk=0, weights="softmax", head_bias=None, keep_first=0):
+                        plan=None, softcap=0.0, chunk=0, weights="softmax", head_bias=None, keep_first=0, value_cols=None):
         """Causal attention of the step's query rows over the paged keys and values.  ``window`` > 0: a row at position p
         sees keys p - window + 1 .. p, and with ``keep_first`` > 0 also the sequence's first ``keep_first`` keys.  ``chunk`` > 0 (instead of a window): a row at position p sees the keys of its own
         chunk of ``chunk`` positions up to p, chunks counted from position 0 of the sequence.  ``softcap`` > 0: a score s
         (scale applied) becomes softcap * tanh(s / softcap) before mask and softmax.  ``weights`` "sigmoid": a visible key
         weighs sigmoid(score + head_bias[head]) (``head_bias`` float32 [num_heads] or None) and nothing is normalised over the
-        keys; every kernel but the thread-block-cluster decode form computes them."""
+        keys; every kernel but the thread-block-cluster decode form computes them.  ``value_cols`` (n, heads): of a value row
+        only a piece is a head's own, the columns h // heads * n .. + n, and ``out`` is [T, num_heads * n] (tensor-core kernels: n
+        a multiple of 8, of 32 with tcgen05)."""
         if weights not in ("softmax", "sigmoid"):
             raise KernelError(f"paged_attention: unknown kind of weights {weights!r}")
         sig = weights == "sigmoid"
@@ -865,27 +879,30 @@ class CudaOps:
             page_size, sig)
         if sig and kernel not in ("mma", "simt", "tc", "tcpp"):
             raise KernelError(f"paged_attention: sigmoid weights have no {kernel!r} kernel")
+        dv, per = value_cols if value_cols is not None else (0, 1)
+        if dv and kernel == "simt":
+            raise KernelError("paged_attention: value columns per head belong to the tensor-core kernels")
         if kernel in ("tc", "tcpp"):
             scratch = None
             if num_splits > 1:
-                scratch = torch.empty((T * num_heads * num_splits * (head_dim + 2),), dtype=torch.float32, device=qkv.device)
+                scratch = torch.empty((T * num_heads * num_splits * ((dv or head_dim) + 2),), dtype=torch.float32, device=qkv.device)
             self._check(self.lib.ttie_paged_attention_tc_weights(
                 _ptr(qkv), qkv.stride(0), _ptr(k_pages), _ptr(v_pages), k_pages.shape[0], _ptr(block_table),
                 block_table.shape[1], page_size, _ptr(query_start_loc), _ptr(seq_lens), _ptr(out), T, num_seqs, num_heads,
                 num_kv_heads, head_dim, max_q_len, float(scale), float(softcap or 0.0), int(window), int(chunk), int(keep_first), num_splits, split_len, _ptr(scratch),
-                1 if kernel == "tcpp" else 0, 1 if sig else 0, _ptr(head_bias), self._stream(qkv)), "paged_attention_tc")
+                1 if kernel == "tcpp" else 0, 1 if sig else 0, _ptr(head_bias), dv, per, 0, self._stream(qkv)), "paged_attention_tc")
             self.launches += 2 if num_splits > 1 else 1
             return
         form = {"mma": 0, "mma_c2": 2, "mma_c4": 4}.get(kernel)
         scratch = None
         if num_splits > 1 and not form:
-            scratch = torch.empty((T * num_heads * num_splits * (head_dim + 2),), dtype=torch.float32, device=qkv.device)
+            scratch = torch.empty((T * num_heads * num_splits * ((dv or head_dim) + 2),), dtype=torch.float32, device=qkv.device)
         if form is not None:
             self._check(self.lib.ttie_paged_attention_mma_weights(
                 _ptr(qkv), qkv.stride(0), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1],
                 page_size, _ptr(query_start_loc), _ptr(seq_lens), _ptr(out), T, num_seqs, num_heads, num_kv_heads,
                 head_dim, max_q_len, float(scale), float(softcap or 0.0), int(window), int(chunk), int(keep_first), num_splits, split_len, _ptr(scratch),
-                form, 1 if sig else 0, _ptr(head_bias), self._stream(qkv)), "paged_attention_mma")
+                form, 1 if sig else 0, _ptr(head_bias), dv, per, self._stream(qkv)), "paged_attention_mma")
             self.launches += 2 if (num_splits > 1 and not form) else 1
             return
         else:
@@ -946,7 +963,16 @@ class CudaOps:
 
     def joint_plan(self, dtype, num_seqs, num_heads, kv_heads, width, v_dim, max_q_len, max_kv_len, page_size, keep_first=0):
         """(kernel, num_splits, split_len) for attention over joint rows: a tensor-core kernel that sees one shared key head of
-        ``width`` values where one takes that width, else "joint", the general kernel."""
+        ``width`` values where one takes that width ("tcpg": the two-tile tcgen05 kernel with the rows of one kv head's heads per
+        tile, whose products with the values then have that kv head's columns only), else "joint", the general kernel."""
+        per = num_heads // kv_heads
+        if (dtype == torch.bfloat16 and width in (128, 256) and v_dim in (64, 128) and (kv_heads > 1 or v_dim < width)
+                and max_q_len * per >= self.attn_tc_min_rows and self.lib.ttie_attn_tc_supported(width, page_size)):
+            base = num_seqs * kv_heads * math.ceil(max_q_len * per / 256)
+            if base > self.num_sms // 2:
+                return "tcpg", 1, 0
+            return self._portion_pieces(num_seqs * num_heads * max_q_len, v_dim, max_kv_len,
+                                        (("tcpg", base, 0.017 * (width + v_dim) / 256),), max_kv_len >= 2 * max_q_len)
         if dtype == torch.bfloat16 and (self.lib.ttie_attn_mma_supported(width)
                                         or (width > 128 and self.lib.ttie_attn_tc_supported(width, page_size))):
             return self.attention_plan(dtype, num_seqs, num_heads, 1, width, max_q_len, max_kv_len, page_size)
@@ -968,11 +994,23 @@ class CudaOps:
         kernel, num_splits, split_len = plan if plan is not None else self.joint_plan(
             q.dtype, num_seqs, num_heads, kv_heads, width, v_dim, max_q_len, self.visible_keys(max_q_len, max_kv_len, window, chunk, keep_first),
             page_size)
+        per = num_heads // kv_heads
+        if kernel == "tcpg":
+            scratch = torch.empty((T * num_heads * num_splits * (v_dim + 2),), dtype=torch.float32, device=q.device) if num_splits > 1 else None
+            self._check(self.lib.ttie_paged_attention_tc_weights(
+                _ptr(q), q.stride(0), _ptr(k_pages), _ptr(v_pages), k_pages.shape[0], _ptr(block_table), block_table.shape[1], page_size,
+                _ptr(query_start_loc), _ptr(seq_lens), _ptr(out), T, num_seqs, num_heads, kv_heads, width, max_q_len, float(scale), 0.0,
+                int(window), int(chunk), int(keep_first), num_splits, split_len, _ptr(scratch), 1, 0, None, 0, 1, v_dim, self._stream(q)),
+                "paged_attention_tc (joint rows)")
+            self.launches += 2 if num_splits > 1 else 1
+            return
         if kernel != "joint":
-            direct = kv_heads == 1 and v_dim == width
+            whole = kv_heads == 1 and v_dim == width
+            direct = whole or v_dim % (32 if kernel in ("tc", "tcpp") else 8) == 0     # the kernel itself keeps each head's own columns
             rows = out if direct else torch.empty((T, num_heads * width), dtype=q.dtype, device=q.device)
             self.paged_attention(q, num_heads, 1, width, k_pages, v_pages, block_table, page_size, query_start_loc, seq_lens, num_seqs,
-                                 max_q_len, max_kv_len, scale, window, rows, plan=(kernel, num_splits, split_len), chunk=chunk, keep_first=keep_first)
+                                 max_q_len, max_kv_len, scale, window, rows, plan=(kernel, num_splits, split_len), chunk=chunk, keep_first=keep_first,
+                                 value_cols=(v_dim, per) if direct and not whole else None)
             if not direct:
                 self._check(self.lib.ttie_joint_values(_ptr(rows), _ptr(out), T, num_heads, kv_heads, v_dim, width, self._dt(q), self._stream(q)),
                             "joint_values")
@@ -1128,7 +1166,7 @@ class CudaOps:
         return out
 
     # ---- selective scan
-    selective_warps = 12                    # warps per SM (4 schedulers) that a long prompt's scan is cut into parts for,
+    selective_warps = 56                    # warps per SM, resident or not, that a long prompt's scan is cut into parts for,
     selective_max_parts = 16                # at most this many a request,
     selective_part_tokens = 64              # of at least this many tokens
 
@@ -1136,20 +1174,17 @@ class CudaOps:
         """Into how many parts a request's tokens are walked: every part but the last is walked twice, which pays while the
         channels alone give the SMs too few warps to hide a token's latency."""
         longest = num_tokens - (num_seqs - 1)                          # the most tokens one request of the step can bring
-        pad = self.selective_state_pad(states)
-        lanes = pad // (4 if states <= 128 else 8 if states <= 256 else 16)
+        lanes = self.selective_state_pad(states) // 4
         warps = num_seqs * -(-channels * lanes // 32)
         return max(1, min(self.selective_max_parts, longest // self.selective_part_tokens, self.selective_warps * self.num_sms // warps))
 
     @staticmethod
     def selective_state_pad(states: int) -> int:
-        """States of a channel's row as the scan lays it out: a power-of-two number of slices of 4 (up to 128 states), 8 (up to
-        256) or 16."""
-        per_thread = 4 if states <= 128 else 8 if states <= 256 else 16
-        slices = 1
-        while slices * per_thread < states:
-            slices *= 2
-        return slices * per_thread
+        """States of a channel's row as the scan lays it out: a power-of-two number of slices of 4."""
+        pad = 4
+        while pad < states:
+            pad *= 2
+        return pad
 
     def selective_scan(self, u, dt, dt_bias, A, D, bc, col_b, col_c, z, state, xin, tail, taps, query_start_loc, slot_ids, num_seqs, states):
         """The diagonal recurrence over the step's tokens from the state rows ``state`` [slots + 1, channels, padded states] (advanced

@@ -23,17 +23,15 @@ import torch
 from .base import Mixer, ParamSpec, FixedStateNeed, StepContext
 from ..registry import register_part
 
-MAX_STATES = 512                # states per channel the scan kernel takes (csrc/selective_scan.cu)
+MAX_STATES = 128                # states per channel the scan kernel takes (csrc/selective_scan.cu)
 
 
 def padded_states(states: int) -> int:
-    """States of a channel's row as the scan kernel lays it out: a power-of-two number of slices of 4 (up to 128 states), 8 (up
-    to 256) or 16."""
-    per_thread = 4 if states <= 128 else 8 if states <= 256 else 16
-    slices = 1
-    while slices * per_thread < states:
-        slices *= 2
-    return slices * per_thread
+    """States of a channel's row as the scan kernel lays it out: a power-of-two number of slices of 4."""
+    pad = 4
+    while pad < states:
+        pad *= 2
+    return pad
 
 
 def _up8(n: int) -> int:
@@ -100,7 +98,7 @@ class SelectiveScan(Mixer):
         u32, u_c = ops.causal_conv(proj, 0, I, self.taps, self.conv_w, self.conv_b, tail, ctx.token_seq, ctx.query_start_loc, ctx.slot_ids,
                                    lowp, first_row=0, act="silu", want_f32=not lowp)
         u = u_c if lowp else u32
-        low = ops.linear(u, self.w_x, None)                                                    # [T, d | B | C]
+        low = ops.linear_narrow(u, self.w_x)                                                  # [T, d | B | C]
         dt = ops.linear(low[:, :self.w_dt.shape[1]], self.w_dt, None, out_dtype=torch.float32)  # [T, inner] float32
         y = ops.selective_scan(u, dt, self.dt_b, self.A, self.D, low, self.col_b, self.col_c, proj[:, I:], S, proj, tail, self.taps,
                                ctx.query_start_loc, ctx.slot_ids, ctx.num_seqs, self.state)
