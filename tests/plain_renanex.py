@@ -130,7 +130,8 @@ def mixed_scores(q, k, talk, scale):
 
 def attention(h, W, p, m, eps, shared):
     S = h.shape[0]
-    H, G, D, Dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    H, D = m["heads"], m["dim"]
+    G, Dv = m.get("kv_heads", H), m.get("vdim", D)
     q = rms_norm(h @ W[p + "q"].T, eps, W[p + "q.norm"])
     k = rms_norm(h @ W[p + "k"].T, eps, W[p + "k.norm"])
     v = h @ W[p + "v"].T
