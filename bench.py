@@ -352,12 +352,12 @@ def dabilorn_config(width, heads, layers=4):
 def renanex_config(width, heads, layers=4):
     """A Renanex model at layer sizes that resemble a real model's: selective scan with twice the width as channels, 16 states, a
     step-size rank of width / 16 and four convolution taps; linear attention with width / 128 heads of 128 key and 128 value
-    channels; attention with scores mixed over the heads, heads of 128 on one kv head (two from 16 heads on), YaRN-rescaled
+    channels; attention with scores mixed over the heads, heads of 128 (eight query heads per kv head), YaRN-rescaled
     rotation, a window of 1,024 keys that keeps the first four, and blended values; feed-forwards of 4 x width.  Layer order:
     selective scan, linear attention, attention, attention, repeated."""
     ssm = {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}
     lin = {"heads": heads, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5 - 3 * i / max(1, heads - 1)) for i in range(heads)]}
-    att = {"heads": heads, "kv_heads": 2 if heads >= 16 else 1, "dim": 128, "vdim": 128, "mask": {"size": 1024, "keep_first": 4},
+    att = {"heads": heads, "kv_heads": max(1, heads // 8), "dim": 128, "vdim": 128, "mask": {"size": 1024, "keep_first": 4},
            "rot": {"base": 10000.0, "dims": 128, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}},
            "scale": 128 ** -0.5, "v_mix": True}
     ff = {"kind": "dense", "ff": 4 * width}

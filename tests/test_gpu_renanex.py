@@ -347,7 +347,8 @@ def test_attention_at_other_sizes(ops, dtype, heads, kv_heads, dim, vdim, rot):
 
 @pytest.mark.parametrize("page", [16, 64])
 @pytest.mark.parametrize("window,keep", [(None, None), (200, 4), (333, 150), (64, 64)])
-@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(8, 1, 128, 128), (16, 2, 64, 64), (8, 2, 128, 128), (4, 4, 64, 64), (8, 2, 120, 64), (16, 2, 32, 32)])
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(8, 1, 128, 128), (16, 2, 64, 64), (8, 2, 128, 128), (4, 4, 64, 64), (8, 2, 120, 64), (16, 2, 32, 32), (16, 4, 128, 128),
+                                                      (8, 8, 64, 64), (12, 3, 128, 64)])
 def test_attention_on_the_tensor_core_kernels(ops, heads, kv_heads, dim, vdim, window, keep, page):
     """Pages of 16 and 64 keys and joint rows of 64, 128 and 256 values in bfloat16: prompt portions of several hundred rows take the
     tcgen05 kernels (two query tiles per CTA, per kv head where there are several), decoded tokens behind a long cache take the

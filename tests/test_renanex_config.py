@@ -75,8 +75,8 @@ def test_cache_needs():
 def test_joint_rows_are_padded_to_what_the_kernels_take():
     width = lambda dtype, *a: CudaOps.joint_width(None, dtype, *a)
     bf = torch.bfloat16
-    assert [width(bf, *a) for a in ((2, 24, 8), (2, 10, 12), (1, 128, 64), (2, 65, 8), (3, 80, 90), (8, 64, 64), (3, 87, 1))] == \
-        [48, 32, 128, 256, 272, 512, 264]
+    assert [width(bf, *a) for a in ((2, 24, 8), (2, 10, 12), (1, 128, 64), (2, 65, 8), (3, 80, 90), (8, 64, 64), (3, 87, 1), (4, 100, 128), (5, 100, 100))] == \
+        [48, 32, 128, 256, 272, 512, 264, 512, 504]
     assert width(torch.float32, 3, 7, 5) == 24 and width(torch.float32, 1, 6, 30) == 32
 
 

@@ -101,10 +101,10 @@ def simulate(nsteps, ntq, seed, product_barriers_per_tile=2, softmax_threads=2, 
         for j in range(nsteps):
             b, par, idx = j & 1, (j >> 1) & 1, v_index(j)
             st = idx % NS
-            yield from wait(("FULL", st), (idx // NS) & 1)
-            assert ring[st] == ("V", j), ("values from the wrong tile", j, ring[st])
             yield from wait(("PF", t, b), par)
             yield from wait(("OC", t, b), par)
+            yield from wait(("FULL", st), (idx // NS) & 1)
+            assert ring[st] == ("V", j), ("values from the wrong tile", j, ring[st])
             for w in range(W):
                 assert probs.get((t, b, w)) == j, ("probabilities of another step", t, j)
             pv_issued[t] = j
@@ -193,12 +193,12 @@ def test_protocol_holds_under_random_schedules(nsteps, ntq):
         simulate(nsteps, ntq, seed)
 
 
-@pytest.mark.parametrize("stages,key_entries", [(4, 1), (5, 2)])
+@pytest.mark.parametrize("stages,key_entries", [(4, 1), (5, 2), (5, 4)])
 @pytest.mark.parametrize("nsteps", [1, 2, 3, 5, 8, 21])
 def test_protocol_holds_with_short_rings(nsteps, stages, key_entries):
-    """Wide key rows leave room for four entries only, or for five of half a key tile."""
+    """Wide key rows leave room for four entries only, or for five of half or a quarter of a key tile."""
     for ntq in (1, 2):
-        for seed in range(25):
+        for seed in range(60):
             simulate(nsteps, ntq, seed, NS=stages, KE=key_entries)
 
 

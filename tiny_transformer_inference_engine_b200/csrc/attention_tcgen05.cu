@@ -651,10 +651,10 @@ constexpr int NS = 8;                                            // stages of th
 enum { PP_FULL = 0, PP_EMPTY = NS, PP_SF = 2 * NS, PP_PF = PP_SF + 4, PP_SC = PP_PF + 4, PP_OC = PP_SC + 4, PP_OF = PP_OC + 4,
        PP_LF = PP_OF + 4, PP_NBARS = PP_LF + 2 };                // SF, PF, SC, OC, OF: [tile][step parity]
 constexpr int PP_NTHREADS = 512;
-// What 227 KB leave beside NT query tiles: with two tiles of 256-column rows a key tile travels as two entries of the ring (128
-// columns each), so that five entries of 16 KB fit.
-__host__ __device__ constexpr int key_entries(int D, int NT) { return D > 128 && NT > 1 ? 2 : 1; }
-__host__ __device__ constexpr int ring_stages(int D, int NT) { return D > 128 ? (NT > 1 ? 5 : 4) : NS; }
+// What 227 KB leave beside NT query tiles: with two tiles of 256-column rows, or one of 512, a key tile travels as two or four
+// entries of the ring (128 columns each), so that five entries of 16 KB fit.
+__host__ __device__ constexpr int key_entries(int D, int NT) { return D > 256 ? 4 : D > 128 && NT > 1 ? 2 : 1; }
+__host__ __device__ constexpr int ring_stages(int D, int NT) { return key_entries(D, NT) > 1 ? 5 : D > 128 ? 4 : NS; }
 __host__ __device__ constexpr int entry_blocks(int D, int DO, int NT) {          // 64-column blocks of an entry
     return D / 64 / key_entries(D, NT) > DO / 64 ? D / 64 / key_entries(D, NT) : DO / 64;
 }
@@ -683,7 +683,7 @@ __device__ __forceinline__ void tmem_st32(uint32_t taddr, const uint32_t (&r)[32
 
 // D: key size; DO: value columns (D, or fewer: the value columns of one kv head of a joint row).  NT: query tiles per CTA.  Tensor
 // memory holds 2 x 2 x 64 score columns and NT x DO output columns: two tiles up to 128 output columns, one tile (its scores
-// at columns 0..127, its output at 256..511) at 256.
+// at columns 0..127, its output at 256..511) at 256, and one at 512 key columns, where shared memory holds one query tile.
 template <int D, int DO, int NT>
 __global__ void __launch_bounds__(pp::PP_NTHREADS, 1)
 attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const AttnTcParams p) {
@@ -1070,9 +1070,11 @@ attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
                 for (int j = 0; j < nsteps; ++j) {
                     const int b = j & 1, idx = v_index(j), st = idx % NSD;
                     const uint32_t par = (j >> 1) & 1;
-                    if (!mbar_wait(BAR(PP_FULL + st), (idx / NSD) & 1, 5)) break;
+                    // the copy is waited for last: with P there its keys were, so the entry's barrier is at most a phase behind
+                    // (short rings: on its first lap a wait for the second lap's parity would pass)
                     if (!mbar_wait(BAR(PP_PF + 2 * t + b), par, 7)) break;
                     if (!mbar_wait(BAR(PP_OC + 2 * t + b), par, 6)) break;
+                    if (!mbar_wait(BAR(PP_FULL + st), (idx / NSD) & 1, 5)) break;
                     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                     const uint32_t v_lo = ring_v_lo + (uint32_t)st * (KV_BYTES >> 4);
                     const uint32_t p_tmem = s_tmem + (uint32_t)b * BNK;      // P sits where the step's scores sat
@@ -1161,7 +1163,7 @@ int launch(const CUtensorMap& mk, const CUtensorMap& mv, const AttnTcParams& p, 
 }
 template <int D, int DO>
 int launch_pp(const CUtensorMap& mk, const CUtensorMap& mv, const AttnTcParams& p, cudaStream_t s) {
-    constexpr int NT = DO > 128 ? 1 : 2, NSD = pp::ring_stages(D, NT);
+    constexpr int NT = DO > 128 || D > 256 ? 1 : 2, NSD = pp::ring_stages(D, NT);
     const size_t smem = NT * (size_t)(D / 64) * BM * 128 + NSD * (size_t)pp::entry_blocks(D, DO, NT) * pp::BNK * 128 + 1024;
     auto k = attn_tc_pp_kernel<D, DO, NT>;
     static bool allowed[64] = {false};                           // the attribute is set once per device
@@ -1218,6 +1220,11 @@ extern "C" int ttie_attn_tc_supported(int D, int page_size) {
     return (D == 64 || D == 128 || D == 256) && page_size >= 8 && page_size % 8 == 0 && (128 % page_size == 0 || page_size % 128 == 0) && page_size <= 256;
 }
 
+// Joint rows with a row group per kv head: rows of 128, 256 or 512 values, kv heads of 64 or 128 value columns.
+extern "C" int ttie_attn_tc_joint_supported(int W, int dv, int page_size) {
+    return (W == 128 || W == 256 || W == 512) && (dv == 64 || dv == 128) && ttie_attn_tc_supported(128, page_size);
+}
+
 // two_tiles: 0 = a CTA owns one 128-row query tile (any number of rows; decode steps; head size 64 or 128), 1 = the
 // kernel for prompt portions: a CTA owns 256 rows as two tiles taken in turns (128 rows as one tile at head size 256).
 // num_splits > 1: the key range is cut into pieces of split_len keys (a multiple of 128) over grid y; the partial
@@ -1249,7 +1256,7 @@ extern "C" int ttie_paged_attention_tc_weights(const void* q, long long q_stride
                                                float* scratch, int two_tiles, int weights, const float* head_bias, int dv, int per, int joint, void* stream) {
     if (T <= 0 || num_seqs <= 0) return 0;
     if (weights != 0 && weights != 1) TTIE_FAIL("attention_tc: unknown kind of weights %d", weights);
-    if (!ttie_attn_tc_supported(D, page_size)) TTIE_FAIL("attention_tc: head size %d with pages of %d keys is not supported", D, page_size);
+    if (!joint && !ttie_attn_tc_supported(D, page_size)) TTIE_FAIL("attention_tc: head size %d with pages of %d keys is not supported", D, page_size);
     if (Hkv <= 0 || Hq % Hkv) TTIE_FAIL("attention_tc: %d heads are not a multiple of %d kv heads", Hq, Hkv);
     if (q_stride % 8 || ((uintptr_t)q | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)out | (uintptr_t)scratch) & 15)
         TTIE_FAIL("attention_tc: pointers must be 16-byte aligned and the query stride a multiple of 8");
@@ -1260,7 +1267,7 @@ extern "C" int ttie_paged_attention_tc_weights(const void* q, long long q_stride
     if (num_splits > 65535) TTIE_FAIL("attention_tc: too many splits (%d)", num_splits);
     CUtensorMap mk, mv;
     if (dv > 0 && (dv % 32 || per <= 0 || (long long)ceil_div(Hq, per) * dv > D)) TTIE_FAIL("attention_tc: %d value columns per %d heads in rows of %d", dv, per, D);
-    if (joint && (!two_tiles || (joint != 64 && joint != 128) || (D != 128 && D != 256) || (long long)Hkv * joint > D))
+    if (joint && (!two_tiles || !ttie_attn_tc_joint_supported(D, joint, page_size) || (long long)Hkv * joint > D))
         TTIE_FAIL("attention_tc: %d kv heads of %d value columns in joint rows of %d are not supported", Hkv, joint, D);
     const long long rows = (long long)num_pages * (joint ? 1 : Hkv) * page_size;
     const int tile_keys = two_tiles ? pp::BNK : BN;              // keys per copy tile of the kernel
@@ -1273,7 +1280,7 @@ extern "C" int ttie_paged_attention_tc_weights(const void* q, long long q_stride
     p.num_seqs = num_seqs; p.Hq = Hq; p.Hkv = Hkv; p.scale_log2 = scale * 1.4426950408889634f; p.window = window; p.chunk = chunk;
     p.keep = window > 0 ? keep : 0;
     p.cap_in = softcap > 0.f ? scale / softcap : 0.f; p.cap_out = softcap > 0.f ? softcap / scale : 0.f;
-    p.row_tiles = ceil_div(max_q_len * (Hq / Hkv), two_tiles && (D <= 128 || joint) ? 2 * BM : BM);
+    p.row_tiles = ceil_div(max_q_len * (Hq / Hkv), two_tiles && (D <= 128 || (joint && D <= 256)) ? 2 * BM : BM);
     p.num_splits = num_splits; p.split_len = split_len;
     p.sigmoid = weights; p.head_bias = head_bias;
     p.dv = dv; p.per = per > 0 ? per : 1; p.joint = joint ? 1 : 0;
@@ -1284,7 +1291,8 @@ extern "C" int ttie_paged_attention_tc_weights(const void* q, long long q_stride
     const int rows_most = max_q_len * (Hq / Hkv);
     const bool ahead = rows_most >= BM;                          // full row tiles: a prompt portion
     p.q_rows = ahead ? BM : 32 * ceil_div(rows_most, 32);
-    const int rc = joint ? (D == 256 ? (joint == 128 ? launch_pp<256, 128>(mk, mv, p, s) : launch_pp<256, 64>(mk, mv, p, s))
+    const int rc = joint ? (D == 512 ? (joint == 128 ? launch_pp<512, 128>(mk, mv, p, s) : launch_pp<512, 64>(mk, mv, p, s)) :
+                            D == 256 ? (joint == 128 ? launch_pp<256, 128>(mk, mv, p, s) : launch_pp<256, 64>(mk, mv, p, s))
                                      : (joint == 128 ? launch_pp<128, 128>(mk, mv, p, s) : launch_pp<128, 64>(mk, mv, p, s)))
                  : two_tiles ? (D == 64 ? launch_pp<64, 64>(mk, mv, p, s) : D == 128 ? launch_pp<128, 128>(mk, mv, p, s) : launch_pp<256, 256>(mk, mv, p, s))
                  : D == 64 ? (ahead ? launch<64, true, 2>(mk, mv, p, s) : launch<64, false, 4>(mk, mv, p, s))

@@ -88,6 +88,7 @@ _SIGNATURES = {
                              _c_int, _c_void],
     "ttie_joint_values": [_c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void],
     "ttie_attn_joint_tile_rows": [_c_int, _c_int],
+    "ttie_attn_tc_joint_supported": [_c_int, _c_int, _c_int],
     "ttie_paged_attention_joint": [_c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int,
                                    _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int, _c_void],
     "ttie_sum_partials": [_c_void, _c_int, _c_ll, _c_void, _c_ll, _c_int, _c_void],
@@ -926,13 +927,16 @@ class CudaOps:
     # ---- attention whose scores are mixed over the heads: joint rows of all kv heads
     def joint_width(self, dtype, kv_heads, head_dim, v_dim) -> int:
         """Values of a joint key / value row: room for all kv heads' keys and for their values, padded to what the attention
-        kernels take (bfloat16: multiples of 16 up to 128, then 256, else multiples of 8; float32: multiples of 4)."""
+        kernels take (bfloat16: multiples of 16 up to 128, then 256, then 512 where a head's values are 64 or 128, else multiples
+        of 8; float32: multiples of 4)."""
         need = kv_heads * max(head_dim, v_dim)
         if dtype == torch.float32:
             return -(-need // 4) * 4
         if need <= 128:
             return -(-need // 16) * 16
-        return 256 if need <= 256 else -(-need // 8) * 8
+        if need <= 256:
+            return 256
+        return 512 if need <= 512 and v_dim in (64, 128) else -(-need // 8) * 8
 
     def check_joint_attention(self, dtype, num_heads, kv_heads, head_dim, v_dim, page_size):
         """Raises unless the joint-row kernels take the sizes."""
@@ -966,13 +970,16 @@ class CudaOps:
         ``width`` values where one takes that width ("tcpg": the two-tile tcgen05 kernel with the rows of one kv head's heads per
         tile, whose products with the values then have that kv head's columns only), else "joint", the general kernel."""
         per = num_heads // kv_heads
-        if (dtype == torch.bfloat16 and width in (128, 256) and v_dim in (64, 128) and (kv_heads > 1 or v_dim < width)
-                and max_q_len * per >= self.attn_tc_min_rows and self.lib.ttie_attn_tc_supported(width, page_size)):
-            base = num_seqs * kv_heads * math.ceil(max_q_len * per / 256)
+        rows, tile = max_q_len * per, 128 if width > 256 else 256
+        if (dtype == torch.bfloat16 and (kv_heads > 1 or v_dim < width) and (rows >= self.attn_tc_min_rows or width > 256)
+                and self.lib.ttie_attn_tc_joint_supported(width, v_dim, page_size)):
+            base = num_seqs * kv_heads * math.ceil(rows / tile)
+            if rows <= 128:                                            # decoded tokens at 512 columns
+                return self._one_per_sm_pieces("tcpg", base, max_kv_len, 0.030, waves_min_keys=640)
             if base > self.num_sms // 2:
                 return "tcpg", 1, 0
             return self._portion_pieces(num_seqs * num_heads * max_q_len, v_dim, max_kv_len,
-                                        (("tcpg", base, 0.017 * (width + v_dim) / 256),), max_kv_len >= 2 * max_q_len)
+                                        (("tcpg", base, 0.017 * (width + v_dim) / 256 * tile / 256),), max_kv_len >= 2 * max_q_len)
         if dtype == torch.bfloat16 and (self.lib.ttie_attn_mma_supported(width)
                                         or (width > 128 and self.lib.ttie_attn_tc_supported(width, page_size))):
             return self.attention_plan(dtype, num_seqs, num_heads, 1, width, max_q_len, max_kv_len, page_size)
