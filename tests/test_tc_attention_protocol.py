@@ -193,9 +193,9 @@ def test_protocol_holds_under_random_schedules(nsteps, ntq):
         simulate(nsteps, ntq, seed)
 
 
-@pytest.mark.parametrize("stages,key_entries", [(4, 1), (5, 2), (5, 4)])
+@pytest.mark.parametrize("stages,key_entries", [(4, 1), (5, 2), (5, 4), (11, 4)])
 @pytest.mark.parametrize("nsteps", [1, 2, 3, 5, 8, 21])
-def test_protocol_holds_with_short_rings(nsteps, stages, key_entries):
+def test_protocol_holds_with_other_rings(nsteps, stages, key_entries):
     """Wide key rows leave room for four entries only, or for five of half or a quarter of a key tile."""
     for ntq in (1, 2):
         for seed in range(60):

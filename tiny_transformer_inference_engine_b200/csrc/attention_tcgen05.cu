@@ -648,13 +648,16 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
 namespace pp {
 constexpr int BNK = 64;                                          // keys per step
 constexpr int NS = 8;                                            // stages of the key/value ring (head size 256: 4 of them, of twice the size)
-enum { PP_FULL = 0, PP_EMPTY = NS, PP_SF = 2 * NS, PP_PF = PP_SF + 4, PP_SC = PP_PF + 4, PP_OC = PP_SC + 4, PP_OF = PP_OC + 4,
+constexpr int NS_MOST = 11;                                      // the longest ring of any form
+enum { PP_FULL = 0, PP_EMPTY = NS_MOST, PP_SF = 2 * NS_MOST, PP_PF = PP_SF + 4, PP_SC = PP_PF + 4, PP_OC = PP_SC + 4, PP_OF = PP_OC + 4,
        PP_LF = PP_OF + 4, PP_NBARS = PP_LF + 2 };                // SF, PF, SC, OC, OF: [tile][step parity]
 constexpr int PP_NTHREADS = 512;
 // What 227 KB leave beside NT query tiles: with two tiles of 256-column rows, or one of 512, a key tile travels as two or four
-// entries of the ring (128 columns each), so that five entries of 16 KB fit.
+// entries of the ring (128 columns each), so that five entries of 16 KB fit.  QR: rows of a query tile that are staged - a step of
+// few rows (decoded tokens at 512 columns) stages 32 and has room for eleven entries; the product still reads 128 rows, what
+// it finds past them is the next block or the ring and gives score rows that nobody reads.
 __host__ __device__ constexpr int key_entries(int D, int NT) { return D > 256 ? 4 : D > 128 && NT > 1 ? 2 : 1; }
-__host__ __device__ constexpr int ring_stages(int D, int NT) { return key_entries(D, NT) > 1 ? 5 : D > 128 ? 4 : NS; }
+__host__ __device__ constexpr int ring_stages(int D, int NT, int QR) { return QR < BM ? NS_MOST : key_entries(D, NT) > 1 ? 5 : D > 128 ? 4 : NS; }
 __host__ __device__ constexpr int entry_blocks(int D, int DO, int NT) {          // 64-column blocks of an entry
     return D / 64 / key_entries(D, NT) > DO / 64 ? D / 64 / key_entries(D, NT) : DO / 64;
 }
@@ -684,14 +687,14 @@ __device__ __forceinline__ void tmem_st32(uint32_t taddr, const uint32_t (&r)[32
 // D: key size; DO: value columns (D, or fewer: the value columns of one kv head of a joint row).  NT: query tiles per CTA.  Tensor
 // memory holds 2 x 2 x 64 score columns and NT x DO output columns: two tiles up to 128 output columns, one tile (its scores
 // at columns 0..127, its output at 256..511) at 256, and one at 512 key columns, where shared memory holds one query tile.
-template <int D, int DO, int NT>
+template <int D, int DO, int NT, int QR = BM>
 __global__ void __launch_bounds__(pp::PP_NTHREADS, 1)
 attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const AttnTcParams p) {
     using namespace pp;
     static_assert(256 + NT * DO <= 512, "tensor memory: scores of two tiles, then the output tiles");
-    constexpr int NSD = ring_stages(D, NT), KE = key_entries(D, NT);      // ring entries in use; entries of a key tile
+    constexpr int NSD = ring_stages(D, NT, QR), KE = key_entries(D, NT);      // ring entries in use; entries of a key tile
     constexpr int CB = D / 64, CBK = CB / KE, CBV = DO / 64;     // 64-column blocks of a row, of a key entry, of a value tile
-    constexpr uint32_t QBLK = BM * 128, KVBLK = BNK * 128;       // bytes of one 64-column block of a query / key tile
+    constexpr uint32_t QBLK = QR * 128, KVBLK = BNK * 128;       // bytes of one 64-column block of a query / key tile
     constexpr uint32_t QT_BYTES = CB * QBLK, KV_BYTES = entry_blocks(D, DO, NT) * KVBLK, K_BYTES = CBK * KVBLK, V_BYTES = CBV * KVBLK;
     constexpr uint32_t TMEM_COLS = 512;
     constexpr uint32_t S_COL = 0, O_COL = 256;                   // scores of (tile t, buffer b) at t * 128 + b * 64; output of tile t at 256 + t * DO
@@ -755,7 +758,7 @@ attn_tc_pp_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
     // queries of both tiles -> shared memory in the K-major swizzled operand layout (rows past the end: zeros).  They and
     // the newest pages are the predecessor's output: what stands above ran while that kernel was finishing.
     pdl_wait();
-    for (int c = threadIdx.x; c < ntq * BM * (D / 8); c += PP_NTHREADS) {
+    for (int c = threadIdx.x; c < (QR < BM ? QR : ntq * BM) * (D / 8); c += PP_NTHREADS) {
         const int r = c / (D / 8), chunk = c - r * (D / 8);      // chunk: 8 bfloat16 = 16 bytes
         const int row = row0 + r;
         uint4 v = make_uint4(0u, 0u, 0u, 0u);
@@ -1161,11 +1164,11 @@ int launch(const CUtensorMap& mk, const CUtensorMap& mv, const AttnTcParams& p, 
     TTIE_CHECK_LAUNCH("attention_tc");
     return 0;
 }
-template <int D, int DO>
+template <int D, int DO, int QR = BM>
 int launch_pp(const CUtensorMap& mk, const CUtensorMap& mv, const AttnTcParams& p, cudaStream_t s) {
-    constexpr int NT = DO > 128 || D > 256 ? 1 : 2, NSD = pp::ring_stages(D, NT);
-    const size_t smem = NT * (size_t)(D / 64) * BM * 128 + NSD * (size_t)pp::entry_blocks(D, DO, NT) * pp::BNK * 128 + 1024;
-    auto k = attn_tc_pp_kernel<D, DO, NT>;
+    constexpr int NT = DO > 128 || D > 256 ? 1 : 2, NSD = pp::ring_stages(D, NT, QR);
+    const size_t smem = NT * (size_t)(D / 64) * QR * 128 + NSD * (size_t)pp::entry_blocks(D, DO, NT) * pp::BNK * 128 + 1024;
+    auto k = attn_tc_pp_kernel<D, DO, NT, QR>;
     static bool allowed[64] = {false};                           // the attribute is set once per device
     int dev = 0;
     if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) dev = 0;
@@ -1291,7 +1294,8 @@ extern "C" int ttie_paged_attention_tc_weights(const void* q, long long q_stride
     const int rows_most = max_q_len * (Hq / Hkv);
     const bool ahead = rows_most >= BM;                          // full row tiles: a prompt portion
     p.q_rows = ahead ? BM : 32 * ceil_div(rows_most, 32);
-    const int rc = joint ? (D == 512 ? (joint == 128 ? launch_pp<512, 128>(mk, mv, p, s) : launch_pp<512, 64>(mk, mv, p, s)) :
+    const int rc = joint ? (D == 512 && rows_most <= 32 ? (joint == 128 ? launch_pp<512, 128, 32>(mk, mv, p, s) : launch_pp<512, 64, 32>(mk, mv, p, s)) :
+                            D == 512 ? (joint == 128 ? launch_pp<512, 128>(mk, mv, p, s) : launch_pp<512, 64>(mk, mv, p, s)) :
                             D == 256 ? (joint == 128 ? launch_pp<256, 128>(mk, mv, p, s) : launch_pp<256, 64>(mk, mv, p, s))
                                      : (joint == 128 ? launch_pp<128, 128>(mk, mv, p, s) : launch_pp<128, 64>(mk, mv, p, s)))
                  : two_tiles ? (D == 64 ? launch_pp<64, 64>(mk, mv, p, s) : D == 128 ? launch_pp<128, 128>(mk, mv, p, s) : launch_pp<256, 256>(mk, mv, p, s))
