@@ -445,10 +445,11 @@ def op_cost(name, args, kw, out, kv_lens, window):
         q, v, state, n, H, D, Dv = args[0], args[2], args[4], args[7], args[8], args[9], args[10]
         T = q.shape[0]
         return T * (2 * H * D * 4 + H * Dv * v.element_size() + 4 * H * Dv) + 2 * n * state[0].numel() * 4, ("fp32", 2 * T * 2 * H * D * Dv)
-    if name == "selective_scan":                                   # (u, dt, ..., A, D, bc, ..., z, state, ..., requests, states): an exponential and three multiply-adds per state and token
+    if name == "selective_scan":                                   # (u, dt, ..., A, D, bc, ..., z, state, ..., requests, states): three multiply-adds per state and token and an
+                                                                    # exponential, of which an SM does 16 a clock: it takes the time of eight multiply-adds
         u, bc, z, S, n, N = args[0], args[5], args[8], args[9], args[15], args[16]
         T, I = u.shape
-        return T * (3 * I * u.element_size() + 4 * I + bc.shape[1] * bc.element_size()) + 2 * n * I * N * 4, ("fp32", 2 * T * 3 * I * N)
+        return T * (3 * I * u.element_size() + 4 * I + bc.shape[1] * bc.element_size()) + 2 * n * I * N * 4, ("fp32", 2 * T * 8 * I * N)
     if name == "sandwich_norm":                                    # (resid, delta, ...): the stream read and written (gathered rows: read), the delta read, one row out
         rows = kw.get("num_rows") or args[0].shape[0]
         per = args[0].shape[1] * ((4 if kw.get("rows") is not None else 8) + args[6].element_size())

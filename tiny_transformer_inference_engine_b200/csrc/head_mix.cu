@@ -58,6 +58,14 @@ __device__ __forceinline__ void rotate_rows(float* x, int heads, int D, int rot,
     }
 }
 
+// (d0, d1) += (a0, a1) * b, one instruction (fma.rn.f32x2)
+__device__ __forceinline__ void fma2(float& d0, float& d1, float a0, float a1, float b) {
+    asm("{\n\t.reg .b64 ra, rb, rd;\n\tmov.b64 ra, {%2, %3};\n\tmov.b64 rb, {%4, %4};\n\tmov.b64 rd, {%0, %1};\n\t"
+        "fma.rn.f32x2 rd, ra, rb, rd;\n\tmov.b64 {%0, %1}, rd;\n\t}" : "+f"(d0), "+f"(d1) : "f"(a0), "f"(a1), "f"(b));
+}
+__device__ __forceinline__ void store2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void store2(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
+
 template <typename T>
 __global__ void __launch_bounds__(MIXT) joint_qkv_store_kernel(const JointStoreArgs a) {
     extern __shared__ __align__(16) float smem[];
@@ -109,8 +117,35 @@ __global__ void __launch_bounds__(MIXT) joint_qkv_store_kernel(const JointStoreA
             vp[i] = from_f32<T>(v);
         }
     }
-    // the mixed query rows: thread = column of the joint row, HB output heads at a time
+    // the mixed query rows: thread = column of the joint row (two columns where heads have even sizes), HB output heads at a time
     T* q = reinterpret_cast<T*>(a.q_out) + (size_t)t * a.H * a.W;
+    if (a.D % 2 == 0 && a.W % 2 == 0) {
+        const int half = a.W >> 1, blocks = (h1 - h0 + HB - 1) / HB;
+        for (int e = threadIdx.x; e < half * blocks; e += MIXT) {
+            const int hb = e / half * HB, i = (e % half) * 2;
+            const int c = i / a.D, d = i - c * a.D;                  // kv head of the columns
+            float acc[2][HB];
+#pragma unroll
+            for (int k = 0; k < HB; ++k) acc[0][k] = acc[1][k] = 0.f;
+            if (c < a.G) {
+                const float* qc = qs + (size_t)c * per * a.D + d;
+                const float* mc = ms + (size_t)c * per * mh + hb;
+#pragma unroll 4
+                for (int g = 0; g < per; ++g) {
+                    const float2 qv = *reinterpret_cast<const float2*>(qc + g * a.D);
+                    const float4 m0 = *reinterpret_cast<const float4*>(mc + g * mh), m1 = *reinterpret_cast<const float4*>(mc + g * mh + 4);
+                    fma2(acc[0][0], acc[0][1], m0.x, m0.y, qv.x); fma2(acc[0][2], acc[0][3], m0.z, m0.w, qv.x);
+                    fma2(acc[0][4], acc[0][5], m1.x, m1.y, qv.x); fma2(acc[0][6], acc[0][7], m1.z, m1.w, qv.x);
+                    fma2(acc[1][0], acc[1][1], m0.x, m0.y, qv.y); fma2(acc[1][2], acc[1][3], m0.z, m0.w, qv.y);
+                    fma2(acc[1][4], acc[1][5], m1.x, m1.y, qv.y); fma2(acc[1][6], acc[1][7], m1.z, m1.w, qv.y);
+                }
+            }
+#pragma unroll
+            for (int k = 0; k < HB; ++k)
+                if (h0 + hb + k < h1) store2(q + (size_t)(h0 + hb + k) * a.W + i, acc[0][k], acc[1][k]);
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < a.W; i += MIXT) {
         const int c = i / a.D, d = i - c * a.D;                      // kv head of the column
         for (int hb = 0; hb < h1 - h0; hb += HB) {
