@@ -63,7 +63,7 @@ REN_B = model(97, 50, 3e-4, 0.7, None, [
 REN_C = model(120, 128, 1e-6, 1.0, 20.0, [
     layer("mamba1", mamba(256, 40, 16, 3), 128),
     layer("attention", attn(8, 2, 64, 64, 0.125, window=48, keep=5, rot=16, base=1000.0, v_mix=True), 64),
-    layer("lightning", lightning(4, 64, 32, [0.6, 0.9, 0.97, 0.999])),
+    layer("lightning", lightning(4, 64, 32, [0.5, 0.9, 0.98, 0.998])),
     layer("attention", attn(4, 4, 64, 32, 0.12, window=70, keep=20, rot=64, base=1e5, scaling=yarn(2.0, 128, 16.0, 2.0), v_mix=True), 64),
     layer("attention", attn(4, 1, 64, 64, 0.12, window=33, keep=4, rot=32), 64)])
 

@@ -117,7 +117,7 @@ def test_schedules_against_plain_model(name, dtype):
 def test_a_wider_model_with_long_prompts_on_pages_of_16(dtype):
     """Joint rows of 128 and 256 values on pages of 16 keys (the tcgen05 kernels' sizes), prompts of several hundred tokens, windows
     that no page edge meets: whole (the scans walk long prompts in parts), with a decoded tail, and mixed on a pool without slack."""
-    cfg = model(200, 192, 1e-5, 1.0, 15.0, [
+    cfg = model(200, 224, 1e-5, 1.0, 15.0, [
         layer("attention", attn(8, 2, 64, 64, 0.12, window=150, keep=6, rot=64, base=5e4, v_mix=True), 128),
         layer("mamba1", mamba(384, 16, 12, 4), 128),
         layer("lightning", lightning(3, 64, 64, [0.9, 0.99, 0.999]), 128),
@@ -331,7 +331,7 @@ def test_attention_alone(ops, dtype, window, keep):
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("heads,kv_heads,dim,vdim,rot", [
     (8, 2, 64, 64, 16), (4, 2, 128, 128, 128), (4, 1, 32, 48, 0), (3, 3, 32, 16, 32), (1, 1, 16, 16, 16), (6, 6, 64, 64, 64), (5, 5, 10, 6, 4),
-    (16, 8, 96, 40, 48), (8, 2, 48, 13, 48), (4, 4, 100, 300, 20), (2, 1, 250, 64, 10)])
+    (16, 8, 96, 40, 48), (8, 4, 40, 13, 40), (4, 4, 100, 300, 20), (2, 1, 250, 64, 10)])
 def test_attention_at_other_sizes(ops, dtype, heads, kv_heads, dim, vdim, rot):
     """Joint rows of 16 to 1,200 values: those the tile loop and the decode form take in bfloat16, those the tcgen05 kernels take,
     and those only the general kernel takes; value sizes that are multiples of nothing; one head; one kv head per head."""
