@@ -70,13 +70,15 @@ class CacheGroup:
     @property
     def reach(self):
         """The most keys behind (and including) its own that a token of this group reads: the window, the chunk size,
-        or None for all of them."""
-        return self.need.window if self.need.window is not None else self.need.chunk
+        or None for all of them (the longest chunk, where layers of several chunk sizes read the same pages)."""
+        if self.need.window is not None or self.need.chunk is None:
+            return self.need.window
+        return max(self.need.chunk, *self.need.also_chunks, 0)
 
     def first_needed_page(self, start: int) -> int:
         """First logical page a token at position >= start can still read."""
         if self.need.chunk is not None:
-            return (start - start % self.need.chunk) // self.page_size
+            return min(start - start % c for c in (self.need.chunk, *self.need.also_chunks)) // self.page_size
         if self.window is None:
             return 0
         first_key = max(0, start - self.window + 1)

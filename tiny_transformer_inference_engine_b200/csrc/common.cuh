@@ -100,6 +100,15 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
 // merges split-KV partial results (attention_simt.cu)
 int attn_merge_bf16(const float* ws_o, const float* ws_ml, void* out, int rows, int num_splits, int D, cudaStream_t s);
 
+// The activation of a gated unit's gate, 32-bit.  0: g * sigmoid(alpha * g) (alpha 1: silu); 1: the tanh form of gelu,
+// 0.5 g (1 + tanh(u)) = g / (1 + exp(-2u)) with u = sqrt(2 / pi) (g + 0.044715 g^3).
+__device__ __forceinline__ float gelu_tanh(float g) {
+    return g / (1.0f + expf(-1.5957691216057308f * (g + 0.044715f * g * g * g)));
+}
+__device__ __forceinline__ float gate_act(int act, float alpha, float g) {
+    return act == 1 ? gelu_tanh(g) : g / (1.0f + expf(-alpha * g));
+}
+
 static inline int ceil_div(int a, int b) { return (a + b - 1) / b; }
 
 // multiprocessors of the current device (asked once per device)

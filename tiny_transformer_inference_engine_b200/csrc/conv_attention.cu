@@ -9,7 +9,8 @@
 //                         rows, oldest first, and is zero for a new request); with norm weights every q and k head is divided
 //                         by its root mean square (eps inside the root) and multiplied by a weight per channel that all heads
 //                         share; q and k are rotated at the token's position (pairs (i, i + rot/2) or (2i, 2i + 1); cos/sin
-//                         from the step's table); q is multiplied by 1 + coef * ln(floor((pos + 1) / every) + 1) where a
+//                         from the step's table); optionally every rotated q and k head is then divided by its root mean square
+//                         (no weight); q is multiplied by 1 + coef * ln(floor((pos + 1) / every) + 1) where a
 //                         query temperature is set; q is written as [T, Hq, Dp] and k, v into the pages
 //                         [page, Hkv, slot, Dp]; Dp >= max(D, Dv), the rest zero.  v_from_k: the row has no v columns and a
 //                         value head is the key head as it stands before norm and rotation.
@@ -37,6 +38,8 @@ struct QkvArgs {
     const float* norm_w; float norm_eps;                            // [2][D]: the query heads' weights, then the key heads'; null: no norm
     const float* row_inv;                                           // [T][2]: 1 / rms of the token's whole q and whole k projection (one norm over
                                                                     // all heads at once; norm_w is then [Hq*D + Hkv*D], a weight per channel); null: a norm per head
+    float after_eps;                                                // >= 0: behind the rotation every q and k head is divided by its root mean
+                                                                    // square, no weight, this eps inside the root; < 0: none
     int v_from_k;                                                   // the values are the key heads before norm and rotation
     float qt_coef; int qt_every;                                    // query temperature; every 0: none
     const void* v_first; long long ld_first; float v_mix;           // values become (1 - v_mix) * v + v_mix * v_first; null: as they are
@@ -121,9 +124,15 @@ __global__ void __launch_bounds__(128) qkv_conv_rope_store_kernel(const QkvArgs 
     }
     const float2* cs = a.rot > 0 ? a.cs + (size_t)t * (a.rot >> 1) : nullptr;
     const int pos = a.positions[t];
+    float after = 1.f;                                               // what the rotated head is multiplied by
+    if (a.after_eps >= 0.f && kind != 2) {
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < a.D; i += blockDim.x) { const float v = rotated(row, i, a.rot, a.style, cs); ss = fmaf(v, v, ss); }
+        after = 1.0f / sqrtf(block_sum(ss, red) / (float)a.D + a.after_eps);
+    }
     if (kind == 0) {
         T* q = reinterpret_cast<T*>(a.q_out) + ((size_t)t * a.Hq + h) * a.Dp;
-        const float temp = query_temperature(a, pos);
+        const float temp = query_temperature(a, pos) * after;
         for (int i = threadIdx.x; i < a.Dp; i += blockDim.x)
             q[i] = from_f32<T>(i < a.D ? rotated(row, i, a.rot, a.style, cs) * temp : 0.f);
         return;
@@ -134,7 +143,7 @@ __global__ void __launch_bounds__(128) qkv_conv_rope_store_kernel(const QkvArgs 
     if (kind == 1) {
         T* kp = reinterpret_cast<T*>(a.k_pages) + dst;
         for (int i = threadIdx.x; i < a.Dp; i += blockDim.x)
-            kp[i] = from_f32<T>(i < a.D ? rotated(row, i, a.rot, a.style, cs) : 0.f);
+            kp[i] = from_f32<T>(i < a.D ? rotated(row, i, a.rot, a.style, cs) * after : 0.f);
     } else {
         T* vp = reinterpret_cast<T*>(a.v_pages) + dst;
         const T* vf = a.v_first ? reinterpret_cast<const T*>(a.v_first) + (size_t)t * a.ld_first + (size_t)h * a.Dv : nullptr;
@@ -181,6 +190,14 @@ __device__ __forceinline__ void conv8(const QkvArgs& a, const __nv_bfloat16* __r
     }
 }
 
+// sum over the `lanes` adjacent lanes of a head (a power of two, at most a warp)
+__device__ __forceinline__ float head_sum(float v, int lanes) {
+    const unsigned lane = threadIdx.x & 31u;
+    const unsigned group = lanes >= 32 ? 0xffffffffu : ((1u << lanes) - 1u) << (lane & ~(unsigned)(lanes - 1));
+    for (int o = 1; o < lanes; o <<= 1) v += __shfl_xor_sync(group, v, o);
+    return v;
+}
+
 __global__ void __launch_bounds__(256) qkv_conv_rope_store_vec8_kernel(const QkvArgs a, int T_) {
     TTIE_PDL_ENTRY();
     const int chunks = a.Dp >> 3, units = a.Hq + 2 * a.Hkv;
@@ -215,9 +232,7 @@ __global__ void __launch_bounds__(256) qkv_conv_rope_store_vec8_kernel(const Qkv
             float ss = 0.f;
 #pragma unroll
             for (int i = 0; i < 8; ++i) ss = fmaf(out[i], out[i], ss);
-            const unsigned lane = threadIdx.x & 31u;
-            const unsigned group = chunks >= 32 ? 0xffffffffu : ((1u << chunks) - 1u) << (lane & ~(unsigned)(chunks - 1));
-            for (int o = 1; o < chunks; o <<= 1) ss += __shfl_xor_sync(group, ss, o);
+            ss = head_sum(ss, chunks);
             inv = 1.0f / sqrtf(ss / (float)a.D + a.norm_eps);
         }
         if (inside) {
@@ -253,6 +268,15 @@ __global__ void __launch_bounds__(256) qkv_conv_rope_store_vec8_kernel(const Qkv
                 out[i] = x * c.x - y * c.y; out[i + 1] = x * c.y + y * c.x;
             }
         }
+    }
+    if (a.after_eps >= 0.f && kind != 2) {                           // (values past D are zero and add nothing)
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) ss = fmaf(out[i], out[i], ss);
+        ss = head_sum(ss, chunks);
+        const float after = 1.0f / sqrtf(ss / (float)a.D + a.after_eps);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) out[i] *= after;
     }
     if (kind == 2 && inside && a.v_first) {
         const __nv_bfloat16* vf = reinterpret_cast<const __nv_bfloat16*>(a.v_first) + (size_t)t * a.ld_first + (size_t)h * a.Dv + i0;
@@ -432,7 +456,7 @@ __global__ void gate_head_rows_vec8_kernel(const __nv_bfloat16* __restrict__ att
 extern "C" int ttie_qkv_conv_rope_store(const void* proj, long long ld, int T, int Hq, int Hkv, int D, int Dv, int Dp, int taps,
                                         const float* conv_w, const float* tail, int tail_rows, const int* positions,
                                         const int* token_seq, const int* qsl, const int* slot_ids, const void* cs, int rot, int style,
-                                        const float* norm_w, float norm_eps, const float* row_inv, int v_from_k, float qt_coef, int qt_every,
+                                        const float* norm_w, float norm_eps, const float* row_inv, float after_eps, int v_from_k, float qt_coef, int qt_every,
                                         const void* v_first, long long ld_first, float v_mix, void* q_out, void* k_pages, void* v_pages, const int* block_table, int table_width,
                                         int page_size, int num_pages, int write_kv, int dtype, void* stream) {
     if (T <= 0) return 0;
@@ -446,7 +470,7 @@ extern "C" int ttie_qkv_conv_rope_store(const void* proj, long long ld, int T, i
     QkvArgs a;
     a.proj = proj; a.ld = ld; a.Hq = Hq; a.Hkv = Hkv; a.D = D; a.Dv = Dv; a.Dp = Dp; a.taps = taps; a.conv_w = conv_w; a.tail = tail;
     a.tail_rows = tail_rows; a.positions = positions; a.token_seq = token_seq; a.qsl = qsl; a.slot_ids = slot_ids;
-    a.cs = (const float2*)cs; a.rot = rot; a.style = style; a.norm_w = norm_w; a.norm_eps = norm_eps; a.row_inv = row_inv; a.v_from_k = v_from_k;
+    a.cs = (const float2*)cs; a.rot = rot; a.style = style; a.norm_w = norm_w; a.norm_eps = norm_eps; a.row_inv = row_inv; a.after_eps = after_eps; a.v_from_k = v_from_k;
     a.qt_coef = qt_coef; a.qt_every = qt_every; a.v_first = v_first; a.ld_first = ld_first; a.v_mix = v_mix; a.q_out = q_out; a.k_pages = k_pages; a.v_pages = v_pages;
     a.block_table = block_table; a.table_width = table_width; a.page_size = page_size; a.num_pages = num_pages; a.write_kv = write_kv;
     const size_t smem = (size_t)(D > Dv ? D : Dv) * sizeof(float);
@@ -454,7 +478,7 @@ extern "C" int ttie_qkv_conv_rope_store(const void* proj, long long ld, int T, i
     cudaStream_t s = (cudaStream_t)stream;
     const bool aligned = !(((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)conv_w | (uintptr_t)tail) & 15);
     const int lanes = Dp / 8;                                        // of a head in the eight-values form; a norm adds up over them by shuffles
-    const bool norm_ok = !norm_w || row_inv || (Dp % 8 == 0 && lanes <= 32 && (lanes & (lanes - 1)) == 0);
+    const bool norm_ok = ((!norm_w || row_inv) && after_eps < 0.f) || (Dp % 8 == 0 && lanes <= 32 && (lanes & (lanes - 1)) == 0);
     if (dtype == kBF16 && D % 8 == 0 && Dv % 8 == 0 && Dp % 8 == 0 && ld % 8 == 0 && aligned && norm_ok
         && (rot == 0 || rot % (style == 1 ? 16 : 8) == 0)) {
         const long long threads = (long long)T * (Hq + 2 * Hkv) * (Dp / 8);

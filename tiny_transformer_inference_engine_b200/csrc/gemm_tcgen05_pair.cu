@@ -111,6 +111,7 @@ struct PairParams {
     const __nv_bfloat16* bias;
     int M, N, K;              // N: output columns (SwiGLU: F)
     int up_offset;            // SwiGLU: row of W (and entry of bias) where the up projection starts
+    int gelu;                 // SwiGLU's epilogue with the tanh form of gelu on the gate
     ErrorWords err;           // where a wait that runs out leaves its code
 };
 
@@ -234,7 +235,8 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                             const int col = min(n0 + c * 32 + j, p.N - 1);
                             g += __bfloat162float(p.bias[col]); up += __bfloat162float(p.bias[p.up_offset + col]);
                         }
-                        v[j] = __float_as_uint(g / (1.f + __expf(-g)) * up);
+                        const float z = p.gelu ? 1.5957691216057308f * (g + 0.044715f * g * g * g) : g;
+                        v[j] = __float_as_uint(g / (1.f + __expf(-z)) * up);
                     }
                 } else {
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -308,7 +310,7 @@ int launch(const CUtensorMap& a, const CUtensorMap& b, const PairParams& p, cuda
 
 // C[M,N] = A[M,K] * W[N,K]^T (+ bias) on pairs of CTAs.  A, W bfloat16 with row strides lda, ldw (multiples of 8,
 // 16-byte aligned bases); out_f32 selects float32 output.
-// swiglu != 0: W is [2F, K] (gate rows, then up rows), N = F, C[M, F] = silu(A Wg^T) * (A Wu^T) in bfloat16.
+// swiglu != 0: W is [2F, K] (gate rows, then up rows), N = F, C[M, F] = silu(A Wg^T) * (A Wu^T) in bfloat16 (2: gelu's tanh form instead of silu).
 extern "C" int ttie_gemm_tc_pair(const void* A, long long lda, const void* W, long long ldw, const void* bias, void* C,
                                  long long ldc, int M, int N, int K, int out_f32, int swiglu, void* stream) {
     if (M <= 0 || N <= 0) return 0;
@@ -319,7 +321,7 @@ extern "C" int ttie_gemm_tc_pair(const void* A, long long lda, const void* W, lo
     if (gemm_tc_make_map(&ma, A, M, K, lda, HM)) return -1;
     if (gemm_tc_make_map(&mb, W, swiglu ? 2LL * N : N, K, ldw, HN)) return -1;
     PairParams p;
-    p.C = C; p.ldc = ldc; p.bias = (const __nv_bfloat16*)bias; p.M = M; p.N = N; p.K = K; p.up_offset = swiglu ? N : 0;
+    p.C = C; p.ldc = ldc; p.bias = (const __nv_bfloat16*)bias; p.M = M; p.N = N; p.K = K; p.up_offset = swiglu ? N : 0; p.gelu = swiglu == 2;
     if (gemm_tc_error_words(&p.err.word, &p.err.mirror)) TTIE_FAIL("gemm_tc_pair: the error word's address is not to be had");
     cudaStream_t s = (cudaStream_t)stream;
     // (measured at 2,048 rows: two K blocks per stage with three stages, or seven stages, change nothing - the issuing

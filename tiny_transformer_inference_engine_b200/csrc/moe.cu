@@ -1,6 +1,6 @@
 // Gated linear units with their constants as parameters, and a routed mixture of experts.
 //   glu:            y = g' * sigmoid(alpha * g') * (u' + shift), g' = min(g, limit), u' = clamp(u, -limit, limit) (limit <= 0:
-//                   no clamp); alpha = 1, shift = 0 is SwiGLU.  32-bit arithmetic, rounded once.
+//                   no clamp); alpha = 1, shift = 0 is SwiGLU; act 1: gelu_tanh(g') * (u' + shift).  32-bit arithmetic, rounded once.
 //   moe_route:      scores s = sigmoid(z), or softmax(z) over all experts, from 32-bit router logits; the choice is made by
 //                   c = s + correction (a bias per expert, optional), the weights use s alone; expert e is in group
 //                   e / (E / groups); a group is rated by adding up its `group_top` highest c, the `keep` best-rated
@@ -8,6 +8,7 @@
 //                   weighted s * scale, optionally renormalised to sum to `scale`.  One warp per token, all 32-bit.
 //   moe_plan:       counting sort of the (token, choice) pairs by expert, on the device: offsets per expert, position of each
 //                   pair, and a table of row tiles (expert, first row, rows) for the grouped product; nothing is read on the host.
+//                   The choices come from moe_route or straight from a table that gives each token id its experts.
 //                   Only the first `tile_experts` experts get tiles: the ones behind them are identity experts, which own no
 //                   matrices (their pairs are sorted like the others and no product touches their rows).
 //   grouped_gemm:   C[pos, :] = A[row_of(pos), :] * W[expert_of_tile]^T for every tile of the table (FFMA, 32-bit accumulation,
@@ -21,20 +22,20 @@ namespace {
 
 template <typename T>
 __global__ void glu_kernel(const T* __restrict__ gu, long long ld, T* __restrict__ out, int F, size_t total, float alpha, float limit,
-                           float shift) {
+                           float shift, int act) {
     TTIE_PDL_ENTRY();
     for (size_t e = blockIdx.x * (size_t)blockDim.x + threadIdx.x; e < total; e += (size_t)gridDim.x * blockDim.x) {
         const size_t t = e / F;
         const int f = (int)(e % F);
         float g = to_f32(gu[t * ld + f]), u = to_f32(gu[t * ld + F + f]);
         if (limit > 0.f) { g = fminf(g, limit); u = fminf(fmaxf(u, -limit), limit); }
-        out[e] = from_f32<T>(g / (1.0f + expf(-alpha * g)) * (u + shift));
+        out[e] = from_f32<T>(gate_act(act, alpha, g) * (u + shift));
     }
 }
 
 // bfloat16, 8 values per thread (F and the row stride multiples of 8, 16-byte aligned rows)
 __global__ void glu_vec8_kernel(const __nv_bfloat16* __restrict__ gu, long long ld, __nv_bfloat16* __restrict__ out, int F8, size_t total8,
-                                float alpha, float limit, float shift) {
+                                float alpha, float limit, float shift, int act) {
     TTIE_PDL_ENTRY();
     for (size_t e = blockIdx.x * (size_t)blockDim.x + threadIdx.x; e < total8; e += (size_t)gridDim.x * blockDim.x) {
         const size_t t = e / F8;
@@ -52,7 +53,7 @@ __global__ void glu_vec8_kernel(const __nv_bfloat16* __restrict__ gu, long long 
                 g.x = fminf(g.x, limit); g.y = fminf(g.y, limit);
                 u.x = fminf(fmaxf(u.x, -limit), limit); u.y = fminf(fmaxf(u.y, -limit), limit);
             }
-            o2[i] = __floats2bfloat162_rn(g.x / (1.0f + expf(-alpha * g.x)) * (u.x + shift), g.y / (1.0f + expf(-alpha * g.y)) * (u.y + shift));
+            o2[i] = __floats2bfloat162_rn(gate_act(act, alpha, g.x) * (u.x + shift), gate_act(act, alpha, g.y) * (u.y + shift));
         }
         *reinterpret_cast<uint4*>(out + t * (size_t)F8 * 8 + f) = ov;
     }
@@ -132,14 +133,22 @@ moe_route_kernel(const float* __restrict__ logits, long long ld, int T_, int E, 
 }
 
 // one CTA.  pairs P = T * top.  tiles: int32 [max_tiles][4] = (expert, first row, rows, 0); meta[0] = number of tiles.
+// `table` (int32 [vocab][top], optional): there are no router's choices; the row of a token's id lists its experts.  Otherwise idx[p].
+struct Choices { const int* idx; const int* table; const int* token_ids; int top, vocab, E; };
+__device__ __forceinline__ int expert_of(const Choices& c, int p) {
+    if (!c.table) return c.idx[p];
+    const int t = p / c.top;
+    const int id = min(max(c.token_ids[t], 0), c.vocab - 1);        // ids and entries are validated on the host; never count outside
+    return min(max(c.table[(size_t)id * c.top + (p - t * c.top)], 0), c.E - 1);
+}
 __global__ void __launch_bounds__(1024)
-moe_plan_kernel(const int* __restrict__ idx, int P, int E, int tile_experts, int tile_rows, int max_tiles, int* __restrict__ offsets,
+moe_plan_kernel(const Choices ch, int P, int E, int tile_experts, int tile_rows, int max_tiles, int* __restrict__ offsets,
                 int* __restrict__ pos_of_pair, int* __restrict__ pair_of_pos, int* __restrict__ tiles, int* __restrict__ meta) {
     __shared__ int count[MAX_EXPERTS], cursor[MAX_EXPERTS];
     TTIE_PDL_ENTRY();
     for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
     __syncthreads();
-    for (int p = threadIdx.x; p < P; p += blockDim.x) atomicAdd(&count[idx[p]], 1);
+    for (int p = threadIdx.x; p < P; p += blockDim.x) atomicAdd(&count[expert_of(ch, p)], 1);
     __syncthreads();
     if (threadIdx.x == 0) {
         int at = 0, nt = 0;
@@ -155,7 +164,7 @@ moe_plan_kernel(const int* __restrict__ idx, int P, int E, int tile_experts, int
     }
     __syncthreads();
     for (int p = threadIdx.x; p < P; p += blockDim.x) {
-        const int at = atomicAdd(&cursor[idx[p]], 1);
+        const int at = atomicAdd(&cursor[expert_of(ch, p)], 1);
         pos_of_pair[p] = at;
         pair_of_pos[at] = p;
     }
@@ -416,18 +425,19 @@ __global__ void moe_combine_vec8_kernel(const __nv_bfloat16* __restrict__ Y, con
 inline int grid_for(size_t total) { return (int)((total + 255) / 256 < 8192 ? (total + 255) / 256 : 8192); }
 }  // namespace
 
-extern "C" int ttie_glu(const void* gate_up, long long ld, void* out, int T, int F, float alpha, float limit, float shift, int dtype,
-                        void* stream) {
+extern "C" int ttie_glu(const void* gate_up, long long ld, void* out, int T, int F, float alpha, float limit, float shift, int act,
+                        int dtype, void* stream) {
     if (T <= 0 || F <= 0) return 0;
+    if (act < 0 || act > 1) TTIE_FAIL("glu: unknown activation %d", act);
     const size_t total = (size_t)T * F;
     if (dtype == kBF16 && F % 8 == 0 && ld % 8 == 0 && (((uintptr_t)gate_up | (uintptr_t)out) & 15) == 0) {
         TTIE_LAUNCH(glu_vec8_kernel, grid_for(total / 8), 256, 0, (cudaStream_t)stream, (const __nv_bfloat16*)gate_up, ld, (__nv_bfloat16*)out, F / 8,
-                    total / 8, alpha, limit, shift);
+                    total / 8, alpha, limit, shift, act);
         TTIE_CHECK_LAUNCH("glu");
         return 0;
     }
-    if (dtype == kF32) TTIE_LAUNCH(glu_kernel<float>, grid_for(total), 256, 0, (cudaStream_t)stream, (const float*)gate_up, ld, (float*)out, F, total, alpha, limit, shift);
-    else TTIE_LAUNCH(glu_kernel<__nv_bfloat16>, grid_for(total), 256, 0, (cudaStream_t)stream, (const __nv_bfloat16*)gate_up, ld, (__nv_bfloat16*)out, F, total, alpha, limit, shift);
+    if (dtype == kF32) TTIE_LAUNCH(glu_kernel<float>, grid_for(total), 256, 0, (cudaStream_t)stream, (const float*)gate_up, ld, (float*)out, F, total, alpha, limit, shift, act);
+    else TTIE_LAUNCH(glu_kernel<__nv_bfloat16>, grid_for(total), 256, 0, (cudaStream_t)stream, (const __nv_bfloat16*)gate_up, ld, (__nv_bfloat16*)out, F, total, alpha, limit, shift, act);
     TTIE_CHECK_LAUNCH("glu");
     return 0;
 }
@@ -447,15 +457,24 @@ extern "C" int ttie_moe_route(const float* logits, long long ld, int T, int E, i
     return 0;
 }
 
-extern "C" int ttie_moe_plan(const int* idx, int P, int E, int tile_experts, int max_tiles, int* offsets, int* pos_of_pair, int* pair_of_pos,
-                             int* tiles, int* meta, void* stream) {
+static int launch_plan(const Choices& ch, int P, int E, int tile_experts, int max_tiles, int* offsets, int* pos_of_pair, int* pair_of_pos,
+                       int* tiles, int* meta, cudaStream_t s) {
     if (P <= 0) return 0;
     if (E > MAX_EXPERTS) TTIE_FAIL("moe_plan: %d experts (limit %d)", E, MAX_EXPERTS);
     if (tile_experts < 0 || tile_experts > E) TTIE_FAIL("moe_plan: %d of %d experts own matrices", tile_experts, E);
-    TTIE_LAUNCH(moe_plan_kernel, 1, 1024, 0, (cudaStream_t)stream, idx, P, E, tile_experts, BM, max_tiles, offsets, pos_of_pair, pair_of_pos, tiles,
-                meta);
+    TTIE_LAUNCH(moe_plan_kernel, 1, 1024, 0, s, ch, P, E, tile_experts, BM, max_tiles, offsets, pos_of_pair, pair_of_pos, tiles, meta);
     TTIE_CHECK_LAUNCH("moe_plan");
     return 0;
+}
+extern "C" int ttie_moe_plan(const int* idx, int P, int E, int tile_experts, int max_tiles, int* offsets, int* pos_of_pair, int* pair_of_pos,
+                             int* tiles, int* meta, void* stream) {
+    return launch_plan({idx, nullptr, nullptr, 1, 1, E}, P, E, tile_experts, max_tiles, offsets, pos_of_pair, pair_of_pos, tiles, meta, (cudaStream_t)stream);
+}
+// the experts come from a table of the token ids: table int32 [vocab][top], token_ids int32 [T]
+extern "C" int ttie_moe_plan_table(const int* table, int vocab, const int* token_ids, int T, int top, int E, int max_tiles, int* offsets,
+                                   int* pos_of_pair, int* pair_of_pos, int* tiles, int* meta, void* stream) {
+    if (top < 1 || top > E || vocab < 1) TTIE_FAIL("moe_plan: a table of %d rows with %d of %d experts", vocab, top, E);
+    return launch_plan({nullptr, table, token_ids, top, vocab, E}, T * top, E, E, max_tiles, offsets, pos_of_pair, pair_of_pos, tiles, meta, (cudaStream_t)stream);
 }
 
 // act, row_scale, scale_of: an activation behind an ungated product, see RowAct (act 0 and row_scale null: the plain product)

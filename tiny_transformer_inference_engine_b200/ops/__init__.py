@@ -96,8 +96,12 @@ _SIGNATURES = {
     "ttie_rglru_scan": [_c_void, _c_void, _c_void, _c_void, _c_int, _c_void, _c_void, _c_ll, _c_int, _c_void, _c_ll, _c_int, _c_void,
                         _c_int, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void, _c_int, _c_void,
                         _c_int, _c_void],
-    "ttie_glu": [_c_void, _c_ll, _c_void, _c_int, _c_int, _c_float, _c_float, _c_float, _c_int, _c_void],
+    "ttie_glu": [_c_void, _c_ll, _c_void, _c_int, _c_int, _c_float, _c_float, _c_float, _c_int, _c_int, _c_void],
+    "ttie_residual_sum": [_c_void, _c_void, _c_void, _c_int, _c_ll, _c_void, _c_void, _c_int, _c_ll, _c_void, _c_int, _c_void, _c_int, _c_float,
+                          _c_void, _c_float, _c_void, _c_int, _c_int, _c_int, _c_void],
+    "ttie_token_gate": [_c_void, _c_void, _c_int, _c_ll, _c_void, _c_void, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int, _c_void],
     "ttie_moe_route": [_c_void, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void, _c_void, _c_void, _c_void],
+    "ttie_moe_plan_table": [_c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void],
     "ttie_moe_plan": [_c_void, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void],
     "ttie_grouped_gemm": [_c_void, _c_ll, _c_void, _c_int, _c_void, _c_ll, _c_ll, _c_void, _c_ll, _c_void, _c_void, _c_int, _c_int, _c_int,
                           _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float, _c_void],
@@ -106,11 +110,11 @@ _SIGNATURES = {
     "ttie_row_scale_act": [_c_void, _c_ll, _c_int, _c_int, _c_int, _c_void, _c_void, _c_int, _c_void],
     "ttie_moe_combine_gated": [_c_void, _c_int, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_void, _c_int, _c_void, _c_int, _c_void, _c_ll,
                                _c_void, _c_ll, _c_void],
-    "ttie_skinny_gemm_glu": [_c_void, _c_ll, _c_void, _c_ll, _c_void, _c_ll, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float, _c_void],
+    "ttie_skinny_gemm_glu": [_c_void, _c_ll, _c_void, _c_ll, _c_void, _c_void, _c_ll, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float, _c_int, _c_void],
     "ttie_gather_rows": [_c_void, _c_ll, _c_void, _c_int, _c_int, _c_int, _c_void, _c_int, _c_void],
     "ttie_moe_combine": [_c_void, _c_int, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_void, _c_int, _c_void, _c_int, _c_void, _c_ll, _c_void],
     "ttie_qkv_conv_rope_store": [_c_void, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_int, _c_void,
-                                 _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_float, _c_void, _c_int, _c_float, _c_int,
+                                 _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void, _c_float, _c_void, _c_float, _c_int, _c_float, _c_int,
                                  _c_void, _c_ll, _c_float, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void],
     "ttie_proj_row_rms": [_c_void, _c_ll, _c_int, _c_int, _c_int, _c_float, _c_void, _c_int, _c_void],
     "ttie_stream_conv": [_c_void, _c_int, _c_int, _c_int, _c_void, _c_void, _c_int, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_void],
@@ -469,12 +473,13 @@ class CudaOps:
         self.launches += 1
         return out
 
-    def linear_swiglu_tc_pair(self, x, w_gu, b_gu, hidden):
-        """silu(x @ Wg.T) * (x @ Wu.T) in one kernel: the pair product with the activation in its epilogue."""
+    def linear_swiglu_tc_pair(self, x, w_gu, b_gu, hidden, gate="silu"):
+        """silu(x @ Wg.T) * (x @ Wu.T) in one kernel: the pair product with the activation in its epilogue.  ``gate``
+        "gelu_tanh": gelu's tanh form in place of silu."""
         M, K = x.shape
         act = torch.empty((M, hidden), dtype=torch.bfloat16, device=x.device)
         self._check(self.lib.ttie_gemm_tc_pair(_ptr(x), x.stride(0), _ptr(w_gu), w_gu.stride(0), _ptr(b_gu), _ptr(act), act.stride(0),
-                                               M, hidden, K, 0, 1, self._stream(x)), "gemm_tc_pair (SwiGLU)")
+                                               M, hidden, K, 0, 1 + self._GATE_ACTS[gate], self._stream(x)), "gemm_tc_pair (SwiGLU)")
         self.launches += 1
         return act
 
@@ -1214,7 +1219,8 @@ class CudaOps:
     # ---- attention with a short convolution on its projections, partial rotation, another value size, gated heads
     def qkv_conv_rope_store(self, proj, num_heads, num_kv_heads, head_dim, v_dim, padded_dim, taps, conv_w, tail, positions, token_seq,
                             query_start_loc, slot_ids, cs_table, rot, style, k_pages, v_pages, block_table, page_size, write_kv,
-                            norm_w=None, norm_eps=0.0, v_from_k=False, q_temp=None, row_inv=None, v_first=None, v_mix=0.0):
+                            norm_w=None, norm_eps=0.0, v_from_k=False, q_temp=None, row_inv=None, v_first=None, v_mix=0.0,
+                            norm_after=None):
         """From a step's projected rows ``proj`` [T, >= Hq*D + Hkv*D + Hkv*Dv] (columns [q | k | v]): the short causal
         convolution over time (``conv_w`` float32 tap-major [taps, channels]; ``tail`` float32 state rows
         [slots + 1, taps - 1, channels] with each request's last projected rows; ``taps`` 1 and ``conv_w`` None: none), the
@@ -1227,13 +1233,16 @@ class CudaOps:
         ``row_inv`` (float32 [T, 2] from ``proj_row_rms``): one norm over the whole q and one over the whole k projection
         instead of one per head; ``norm_w`` is then float32 [Hq*D + Hkv*D], a weight per channel.
         ``v_first`` (a view [T, Hkv*Dv] with a row stride): values are stored as (1 - v_mix) * v + v_mix * v_first.
+        ``norm_after`` (its eps): behind the rotation every q and k head is divided by its root mean square, without a weight.
+        ``num_kv_heads`` 0: ``proj`` holds queries only.
         Returns q [T, Hq * padded_dim].  The state rows are advanced by ``conv_tail_update``."""
         T = proj.shape[0]
         q = torch.empty((T, num_heads * padded_dim), dtype=proj.dtype, device=proj.device)
         self._check(self.lib.ttie_qkv_conv_rope_store(
             _ptr(proj), proj.stride(0), T, num_heads, num_kv_heads, head_dim, v_dim, padded_dim, int(taps), _ptr(conv_w), _ptr(tail),
             0 if tail is None else tail.shape[0], _ptr(positions), _ptr(token_seq), _ptr(query_start_loc), _ptr(slot_ids),
-            _ptr(cs_table), int(rot), int(style), _ptr(norm_w), float(norm_eps), _ptr(row_inv), 1 if v_from_k else 0,
+            _ptr(cs_table), int(rot), int(style), _ptr(norm_w), float(norm_eps), _ptr(row_inv),
+            -1.0 if norm_after is None else float(norm_after), 1 if v_from_k else 0,
             float(q_temp[0]) if q_temp else 0.0, int(q_temp[1]) if q_temp else 0,
             _ptr(v_first), 0 if v_first is None else v_first.stride(0), float(v_mix),
             _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1],
@@ -1403,6 +1412,35 @@ class CudaOps:
         self.launches += 1
         return out
 
+    # ---- sub-layers in parallel, a token's own input
+    def residual_sum(self, resid, a, f=None, experts=None, bias=None, mult=1.0, out_dtype=None):
+        """resid <- resid + mult * (a + f + bias) over the 32-bit stream [T, d], in one pass.  ``a``, ``f`` (or None): sub-layers'
+        outputs, [T, d] in the compute dtype or float32, or float32 partial sums [S, T, d]; ``experts`` (rows [P, d], plan, top,
+        weight): plus ``weight`` times the sum of every token's expert rows; ``bias`` float32 [d].  ``out_dtype``: the new rows
+        are also returned in this (the compute) dtype, else None."""
+        T, d = resid.shape
+        out = None if out_dtype is None else torch.empty((T, d), dtype=out_dtype, device=resid.device)
+        terms = [t for t in (a, f) if t is not None]
+        dt = next((t.dtype for t in terms + ([experts[0]] if experts is not None else []) if t.dtype == torch.bfloat16), out_dtype or torch.float32)
+        ap, app, aS, ast = self._delta_args(a)
+        fp, fpp, fS, fst = self._delta_args(f)
+        y, pos, top, weight = (experts[0], experts[1]["pos_of_pair"], int(experts[2]), float(experts[3])) if experts is not None else (None, None, 0, 0.0)
+        self._check(self.lib.ttie_residual_sum(_ptr(resid), ap, app, aS, ast, fp, fpp, fS, fst, _ptr(y), 0 if y is None else self._dt(y), _ptr(pos), top,
+                                               weight, _ptr(bias), float(mult), _ptr(out), T, d, _DT[dt], self._stream(resid)), "residual_sum")
+        self.launches += 1
+        return out
+
+    def token_gate(self, z, token_ids, table, col0, n, dtype):
+        """gelu_tanh(z) * table[token_ids, col0 : col0 + n] -> [T, N] in ``dtype``, zeros in the columns from ``n`` on.  ``z``: [T, N] in
+        the compute dtype, or float32 partial sums [S, T, N]; ``table`` [vocab, columns] in the compute dtype."""
+        T, N = z.shape[-2:]
+        zp, part, S, stride = (None, z.data_ptr(), z.shape[0], z.stride(0)) if z.dim() == 3 else (z.data_ptr(), None, 0, 0)
+        out = torch.empty((T, N), dtype=dtype, device=z.device)
+        self._check(self.lib.ttie_token_gate(zp, part, S, stride, _ptr(token_ids), _ptr(table), table.stride(0), table.shape[0], int(col0), int(n), N, T,
+                                             _ptr(out), self._dt(out), self._stream(out)), "token_gate")
+        self.launches += 1
+        return out
+
     # ---- elementwise functions between products
     _ACTIVATIONS = {"relu2": 0, "tanh": 1, "softcap": 2, "identity": 3, "silu": 4}
 
@@ -1440,12 +1478,15 @@ class CudaOps:
         return self.activation(self.linear(x, w, None), act, inplace=True)
 
     # ---- gated linear units and routed experts
-    def glu(self, gate_up, hidden, alpha=1.0, limit=0.0, shift=0.0):
-        """g * sigmoid(alpha * g) * (u + shift) with optional clamps, gate_up = [g | u] per row -> [T, hidden]."""
+    _GATE_ACTS = {"silu": 0, "gelu_tanh": 1}
+
+    def glu(self, gate_up, hidden, alpha=1.0, limit=0.0, shift=0.0, act="silu"):
+        """g * sigmoid(alpha * g) * (u + shift) with optional clamps, gate_up = [g | u] per row -> [T, hidden].  ``act``
+        "gelu_tanh": the gate passes gelu's tanh form instead (no alpha)."""
         T = gate_up.shape[0]
         out = torch.empty((T, hidden), dtype=gate_up.dtype, device=gate_up.device)
         self._check(self.lib.ttie_glu(_ptr(gate_up), gate_up.stride(0), _ptr(out), T, hidden, float(alpha), float(limit or 0.0),
-                                      float(shift), self._dt(gate_up), self._stream(gate_up)), "glu")
+                                      float(shift), self._GATE_ACTS[act], self._dt(gate_up), self._stream(gate_up)), "glu")
         self.launches += 1
         return out
 
@@ -1479,6 +1520,22 @@ class CudaOps:
         self.launches += 1
         return plan
 
+    def moe_plan_table(self, table, token_ids, num_experts):
+        """``moe_plan`` for experts that a table names: row ``token_ids[t]`` of ``table`` (int32 [vocab, top]) lists token t's
+        experts.  One launch; no choices are written (the plan's ``idx`` is None)."""
+        T, (vocab, top) = token_ids.shape[0], table.shape
+        P = T * top
+        max_tiles = P // int(self.lib.ttie_moe_tile_rows()) + num_experts
+        buf = torch.empty(2 * P + num_experts + 1 + 4 * max_tiles + 4, dtype=torch.int32, device=token_ids.device)
+        plan = {"pos_of_pair": buf[:P], "pair_of_pos": buf[P:2 * P], "offsets": buf[2 * P:2 * P + num_experts + 1],
+                "tiles": buf[2 * P + num_experts + 1:2 * P + num_experts + 1 + 4 * max_tiles], "meta": buf[-4:], "max_tiles": max_tiles,
+                "pairs": P, "idx": None, "real_experts": num_experts}
+        self._check(self.lib.ttie_moe_plan_table(_ptr(table), vocab, _ptr(token_ids), T, top, num_experts, max_tiles, _ptr(plan["offsets"]),
+                                                 _ptr(plan["pos_of_pair"]), _ptr(plan["pair_of_pos"]), _ptr(plan["tiles"]), _ptr(plan["meta"]),
+                                                 self._stream(token_ids)), "moe_plan_table")
+        self.launches += 1
+        return plan
+
     grouped_few_rows = 64                   # (token, choice) pairs up to which the grouped product streams every tile's weights once
 
     def _library_grouped(self, x, w, plan, gather_div):
@@ -1504,20 +1561,26 @@ class CudaOps:
             self._grouped_mm = False                                    # this build has none for the device: the own kernel serves
             return None
 
-    def linear_glu(self, x, w_gu, hidden, alpha=1.0, limit=0.0, shift=0.0):
-        """The gated unit's activation of x @ [Wg; Wu].T -> [M, hidden].  With SwiGLU's constants this is ``linear_swiglu`` and
+    def linear_glu(self, x, w_gu, hidden, alpha=1.0, limit=0.0, shift=0.0, act="silu", bias=None):
+        """The gated unit's activation of x @ [Wg; Wu].T (+ ``bias`` [2 * hidden]) -> [M, hidden].  With SwiGLU's constants this is ``linear_swiglu`` and
         its fused forms; with others, up to 8 rows run the weight-streaming product with the unit in its epilogue (where that
-        form measured faster for the shape), more rows the product and the activation kernel."""
-        if alpha == 1.0 and not limit and shift == 0.0:
-            return self.linear_swiglu(x, w_gu, None, hidden)
-        if x.dtype == torch.bfloat16 and self._skinny_ok(x, w_gu) and self._fused_few_rows_wins(x, w_gu, None, hidden):
-            M, K = x.shape
-            act = torch.empty((M, hidden), dtype=x.dtype, device=x.device)
-            self._check(self.lib.ttie_skinny_gemm_glu(_ptr(x), x.stride(0), _ptr(w_gu), w_gu.stride(0), _ptr(act), hidden, M, hidden, K,
-                                                      float(alpha), float(limit or 0.0), float(shift), self._stream(x)), "skinny_gemm_glu")
+        form measured faster for the shape), more rows the product and the activation kernel; gelu without clamps and shift also has
+        the tcgen05 pair product with the unit in its epilogue (1,024 rows and more, where it measured faster)."""
+        plain = not limit and shift == 0.0
+        if act == "silu" and alpha == 1.0 and plain:
+            return self.linear_swiglu(x, w_gu, bias, hidden)
+        M, K = x.shape
+        if x.dtype == torch.bfloat16 and self._skinny_ok(x, w_gu) and self._fused_few_rows_wins(x, w_gu, bias, hidden):
+            out = torch.empty((M, hidden), dtype=x.dtype, device=x.device)
+            self._check(self.lib.ttie_skinny_gemm_glu(_ptr(x), x.stride(0), _ptr(w_gu), w_gu.stride(0), _ptr(bias), _ptr(out), hidden, M, hidden, K,
+                                                      float(alpha), float(limit or 0.0), float(shift), self._GATE_ACTS[act], self._stream(x)),
+                        "skinny_gemm_glu")
             self.launches += 1
-            return act
-        return self.glu(self.linear(x, w_gu, None), hidden, alpha, limit, shift)
+            return out
+        if (act == "gelu_tanh" and plain and M >= 1024 and x.dtype == torch.bfloat16 and self._skinny_shape_ok(x, w_gu)
+                and self._fused_swiglu_wins(x, w_gu, bias, hidden)):
+            return self.linear_swiglu_tc_pair(x, w_gu, bias, hidden, act)
+        return self.glu(self.linear(x, w_gu, bias), hidden, alpha, limit, shift, act)
 
     def grouped_glu(self, x, w_gu, plan, gather_div, hidden, alpha=1.0, limit=0.0, shift=0.0):
         """The experts' gate/up products over rows sorted by expert, then the gated unit: [pairs, hidden].  Few rows: one

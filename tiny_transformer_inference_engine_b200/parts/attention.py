@@ -31,14 +31,17 @@ only), ``qk_norm`` (its eps: every query and key head is divided by its root mea
 they are cut into heads, and a weight per channel, ``<q><norm_suffix>`` of ``heads * head_dim`` values and ``<k><norm_suffix>`` of
 ``kv_heads * head_dim``; the default ``"head"`` is the norm per head above), ``weights="sigmoid"`` (no softmax: a visible key
 weighs ``sigmoid(score + b_h)`` and the weights are not normalised over the keys; ``head_bias`` names the tensor of one ``b``
-per head, None: no bias), ``keep_first`` (with a window: a token also sees the sequence's first ``keep_first`` tokens, at their true
+per head, None: no bias), ``norm_after`` (its eps: BEHIND the rotation every query and key head is divided by its root mean
+square, without a weight), ``keep_first`` (with a window: a token also sees the sequence's first ``keep_first`` tokens, at their true
 positions), ``v_mix`` (``"first"``: this layer's values are kept for later layers of the step; ``"mix"``: the values become
 ``(1 - l) v + l v_first`` with the number ``l`` of tensor ``v_mix_name`` and ``v_first`` the values of that first layer, and the mixed
 ones are cached), ``head_mix`` (the name of a matrix M [heads, heads]: head h's scores become ``sum_g M[h, g] score_g`` before the
 softmax; see below).  The general step: one product
 ``[W_q; W_k; W_v; W_g] x``; one kernel convolves, normalises, rotates, writes q and stores k and v - rows padded with zeros to
 ``padded_dim``, a multiple of 16 that holds both sizes, so every attention kernel of the package applies; a second moves the
-convolution's inputs into the state row; attention; the gate kernel drops the padding; ``W_o``.
+convolution's inputs into the state row; attention; the gate kernel drops the padding; ``W_o``.  With ``shares_kv`` the general step projects, rotates and norms queries only.
+``cache_chunks``: the chunk sizes (None: no chunks) of the other layers that read this layer's cache, so that a page stays as long as
+any of them needs it.
 
 With ``head_mix`` the mixing goes into the queries: it is linear, so head h's mixed score is the product of ONE query row per head,
 ``[sum of M[h, g] q_g over the heads g of kv head c]`` for every kv head c, with the keys of all kv heads side by side.  One kernel
@@ -67,7 +70,8 @@ class PagedAttention(Mixer):
                  conv_suffix: str = ".conv", chunk: Optional[int] = None, qk_norm: Optional[float] = None,
                  norm_suffix: str = ".norm", v_from_k: bool = False, q_temp: Optional[Dict[str, float]] = None,
                  qk_norm_over: str = "head", weights: str = "softmax", head_bias: Optional[str] = None, keep_first: int = 0,
-                 v_mix: Optional[str] = None, v_mix_name: str = "vmix", head_mix: Optional[str] = None):
+                 v_mix: Optional[str] = None, v_mix_name: str = "vmix", head_mix: Optional[str] = None,
+                 norm_after: Optional[float] = None, cache_chunks=()):
         super().__init__(prefix)
         if num_heads % num_kv_heads:
             raise ValueError(f"num_heads={num_heads} is not a multiple of num_kv_heads={num_kv_heads}")
@@ -133,13 +137,22 @@ class PagedAttention(Mixer):
                                      or self.softcap is not None or self.weights != "softmax" or (self.qk_norm is not None and not self.norm_whole)):
             raise ValueError("scores mixed over the heads exclude a convolution, gates, biases, keys as values, a query temperature, a "
                              "score softcap, other weights than a softmax and a norm per head")
-        self.general = (self.v_head_dim != head_dim or self.v_mix is not None or self.head_mix is not None or self.has_conv or self.gated or self.qkv_bias
+        self.norm_after = None if norm_after is None else float(norm_after)
+        if self.norm_after is not None and head_mix is not None:
+            raise ValueError("scores mixed over the heads exclude a norm behind the rotation")
+        self.cache_chunks = tuple(cache_chunks)
+        if self.cache_chunks and window is not None:
+            raise ValueError("the chunks of other readers of a cache exclude a window of its own layer")
+        self.general = (self.v_head_dim != head_dim or self.norm_after is not None or self.v_mix is not None or self.head_mix is not None or self.has_conv or self.gated or self.qkv_bias
                         or self.rot_dim not in (0, head_dim) or self.qk_norm is not None or self.v_from_k
                         or self.q_temp is not None or self.weights != "softmax")
-        if self.general and (self.shares_kv or self.bias):
-            raise ValueError("the general attention step has neither a shared cache nor an output bias")
+        if self.general and self.bias:
+            raise ValueError("the general attention step has no output bias")
+        if self.general and self.shares_kv and (self.has_conv or self.v_mix is not None or self.norm_whole or self.qk_norm is not None or self.head_mix is not None):
+            raise ValueError("a shared cache excludes a convolution, mixed values, mixed scores and a norm with weights")
         self.padded_dim = -(-max(head_dim, self.v_head_dim) // 16) * 16 if self.general else head_dim
-        self.channels = (num_heads + num_kv_heads) * head_dim + (0 if self.v_from_k else num_kv_heads * self.v_head_dim)   # of [q | k | v]
+        self.proj_kv_heads = 0 if self.shares_kv else num_kv_heads
+        self.channels = (num_heads + self.proj_kv_heads) * head_dim + (0 if self.v_from_k else self.proj_kv_heads * self.v_head_dim)   # of [q | k | v]
         self.conv_w = self.norm_w = None
         self.joint_dim = None                                           # values of a joint cache row (head_mix), set by validate
 
@@ -165,7 +178,9 @@ class PagedAttention(Mixer):
     def _general_specs(self):
         n, d, D, Dv, ws = self.names, self.d_model, self.head_dim, self.v_head_dim, self.weight_suffix
         rows = {"q": self.num_heads * D, "k": self.num_kv_heads * D, "v": self.num_kv_heads * Dv}
-        if self.v_from_k:
+        if self.shares_kv:
+            del rows["k"], rows["v"]
+        elif self.v_from_k:
             del rows["v"]
         specs = {f"{n['o']}{ws}": ParamSpec((d, self.num_heads * Dv))}
         for key, r in rows.items():
@@ -189,7 +204,7 @@ class PagedAttention(Mixer):
 
     def _general_load(self, params):
         n, ws = self.names, self.weight_suffix
-        qkv = ["q", "k"] if self.v_from_k else ["q", "k", "v"]
+        qkv = ["q"] if self.shares_kv else ["q", "k"] if self.v_from_k else ["q", "k", "v"]
         keys = qkv + (["g"] if self.gated else [])
         self.w_in = torch.cat([params[f"{n[k]}{ws}"] for k in keys], dim=0).contiguous()
         self.w_out = params[f"{n['o']}{ws}"].contiguous()
@@ -239,7 +254,12 @@ class PagedAttention(Mixer):
         if self.head_mix is not None:                                   # joint rows: one cache head (its width: validate, or unpadded)
             width = self.joint_dim or self.num_kv_heads * max(self.head_dim, self.v_head_dim)
             return [PagedKVNeed(1, width, self.window, self.page_size, chunk=self.chunk, keep_first=self.keep_first)]
-        needs = [PagedKVNeed(self.num_kv_heads, self.padded_dim, self.window, self.page_size, chunk=self.chunk, keep_first=self.keep_first)]
+        chunk, others = self.chunk, ()
+        if self.cache_chunks:
+            sizes = {self.chunk, *self.cache_chunks}
+            chunk = None if None in sizes else self.chunk
+            others = () if chunk is None else tuple(sorted(sizes - {chunk}))
+        needs = [PagedKVNeed(self.num_kv_heads, self.padded_dim, self.window, self.page_size, chunk=chunk, keep_first=self.keep_first, also_chunks=others)]
         if self.conv_taps > 1:
             needs.append(FixedStateNeed((self.conv_taps - 1, self.channels), "float32"))
         return needs
@@ -297,10 +317,12 @@ class PagedAttention(Mixer):
         state = tail.state if tail is not None else None
         v_first = self._first_values(proj[:, (Hq + Hkv) * D:C], ctx)
         mixed = {} if v_first is None else {"v_first": v_first, "v_mix": self.v_mix_weight}
+        if self.norm_after is not None:
+            mixed["norm_after"] = self.norm_after
         row_inv = ops.proj_row_rms(proj, Hq * D, Hkv * D, self.qk_norm) if self.norm_whole else None
-        q = ops.qkv_conv_rope_store(proj, Hq, Hkv, D, Dv, Dp, self.conv_taps, self.conv_w, state, ctx.positions, ctx.token_seq,
+        q = ops.qkv_conv_rope_store(proj, Hq, self.proj_kv_heads, D, Dv, Dp, self.conv_taps, self.conv_w, state, ctx.positions, ctx.token_seq,
                                     ctx.query_start_loc, ctx.slot_ids, cs, rot, style, cache.k_pages, cache.v_pages,
-                                    cache.block_table, cache.page_size, cache.writable, norm_w=self.norm_w,
+                                    cache.block_table, cache.page_size, cache.writable and not self.shares_kv, norm_w=self.norm_w,
                                     norm_eps=self.qk_norm or 0.0, v_from_k=self.v_from_k, q_temp=self.q_temp, row_inv=row_inv, **mixed)
         if self.conv_taps > 1 and tail.writable:
             ops.conv_tail_update(proj, C, self.conv_taps, state, ctx.query_start_loc, ctx.slot_ids, ctx.num_seqs)

@@ -53,8 +53,8 @@ class ParamSpec:
     """
     shape: Tuple[int, ...]
     storage: str = "matrix"            # "matrix" | "vector" | "table"
-    init: str = "normal"               # random-weights mode: "normal" | "ones" | "zeros"; tables: "randint" | "arange" | "zeros"
-    high: Optional[int] = None         # "randint": values are uniform in [0, high)
+    init: str = "normal"               # random-weights mode: "normal" | "ones" | "zeros"; tables: "randint" | "distinct" | "arange" | "zeros"
+    high: Optional[int] = None         # "randint": values are uniform in [0, high); "distinct": likewise, and differ within a row
     std: Optional[float] = None        # "normal": a standard deviation of this tensor's own (None: the caller's)
 
 
@@ -96,6 +96,7 @@ class PagedKVNeed:
     planes: int = 2                    # 2: keys and values; 1: one array that is both (latent attention), handed out as K and as V
     chunk: Optional[int] = None        # a token reads only keys of its own chunk (chunks counted from position 0); excludes window
     keep_first: int = 0                # with a window: the sequence's first tokens that every later one still reads
+    also_chunks: Tuple[int, ...] = ()  # with a chunk: the chunk sizes of other layers that read these pages; a page stays while any of them reads it
 
 
 @dataclass(frozen=True)

@@ -13,6 +13,7 @@ from typing import Optional
 import torch
 
 from .base import Block, ParamSpec, PartSpec, FixedStateNeed, ResidualStream, StepContext, mixer_cache_argument
+from .moe import ExpertRows
 from ..registry import register_part, build_part
 
 
@@ -179,3 +180,46 @@ class SublayerNormBlock(Block):
         if self.ffn is not None:
             x = self.ffn_norm.add_normed(resid, self.ffn.forward(x, ctx))
         stream.x = x
+
+
+@register_part("block", "parallel")
+class ParallelBlock(Block):
+    """One norm, whose output both sub-layers read, and one sum: ``x = x + mult * (mixer(h) + ffn(h))`` with ``h = norm(x)``; a layer
+    without a feed-forward (``ffn`` None) adds the mixer's output alone.  One kernel forms the sum: it takes the sub-layers'
+    outputs as they leave their last products (partial sums, rows sorted by expert, a bias that the feed-forward left to the block).
+
+    ``side`` and ``side_norm`` (None: neither): a third sub-layer behind that sum which reads the stream itself,
+    ``x = x + side_norm(side(x))``; ``mult`` on it is the norm part's ``gain``.  Its output waits unnormed in ``stream.delta`` with the
+    norm in ``stream.delta_norm``, so the next layer's norm kernel applies that one, adds, and normalises, in one pass."""
+
+    def __init__(self, prefix: str, norm: PartSpec, mixer: PartSpec, ffn: PartSpec = None, mult: float = 1.0, side: PartSpec = None,
+                 side_norm: PartSpec = None):
+        super().__init__(prefix)
+        if (side is None) != (side_norm is None):
+            raise ValueError("a side sub-layer and its norm come together")
+        self.norm = build_part("norm", norm)
+        self.mixer = build_part("mixer", mixer)
+        self.ffn = build_part("ffn", ffn) if ffn is not None else None
+        self.mult = float(mult)
+        self.side = build_part("ffn", side) if side is not None else None
+        self.side_norm = build_part("norm", side_norm) if side_norm is not None else None
+
+    def children(self):
+        return [p for p in (self.norm, self.mixer, self.ffn, self.side, self.side_norm) if p is not None]
+
+    def cache_needs(self):
+        return self.mixer.cache_needs()
+
+    def forward(self, stream: ResidualStream, ctx: StepContext, caches) -> None:
+        ops, resid = self.ops, stream.resid
+        pending = {} if stream.delta_norm is None else {"delta_norm": stream.delta_norm}
+        h = self.norm.add_norm(resid, stream.delta, **pending)
+        a = self.mixer.forward(h, ctx, mixer_cache_argument(self.mixer, caches))
+        f = self.ffn.forward(h, ctx) if self.ffn is not None else None
+        experts = (f.rows, f.plan, f.top, f.weight) if isinstance(f, ExpertRows) else None
+        narrow = self.side is not None and self.dtype != resid.dtype         # the side sub-layer reads the stream in the compute dtype
+        x = ops.residual_sum(resid, a, None if experts is not None else f, experts=experts, bias=getattr(self.ffn, "out_bias", None),
+                             mult=self.mult, out_dtype=self.dtype if narrow else None)
+        stream.delta = stream.delta_norm = None
+        if self.side is not None:
+            stream.delta, stream.delta_norm = self.side.forward(x if narrow else resid, ctx), self.side_norm

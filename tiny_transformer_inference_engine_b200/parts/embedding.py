@@ -2,7 +2,9 @@
 
 Embedding (models/embedding.py:9-15): a row gather, no position term; the gathered row
 (times ``scale``, a parameter; the reference has none) starts the 32-bit residual sum.  ``norm``
-(a norm part's spec; the reference has none): the rows are normed in place before the first layer.  Head (models/transformer_block.py:170,181):
+(a norm part's spec; the reference has none): the rows are normed in place before the first layer.  ``side`` (``name``, ``dim``, ``layers``;
+the reference has none): a second table [vocab, layers * dim] whose row gives every layer its own ``dim`` values of the token; this
+part only owns it and hands it to the step's layers (``TOKEN_SIDE`` in the step's cache of values).  Head (models/transformer_block.py:170,181):
 ``logits = x @ W.T`` without bias, untied from the embedding; logits leave in 32-bit.
 """
 from __future__ import annotations
@@ -13,26 +15,38 @@ from .base import Embedding, Head, ParamSpec, PartSpec, StepContext
 from ..registry import register_part, build_part
 
 
+TOKEN_SIDE = "token side table"          # key of ``StepContext.step_cache``: the table of what a token gives every layer
+
+
 @register_part("embedding", "token")
 class TokenEmbedding(Embedding):
-    def __init__(self, prefix: str, vocab_size: int, dim: int, name: str = "weight", scale: float = 1.0, norm: PartSpec = None):
+    def __init__(self, prefix: str, vocab_size: int, dim: int, name: str = "weight", scale: float = 1.0, norm: PartSpec = None,
+                 side: dict = None):
         super().__init__(prefix)
         self.vocab_size, self.dim, self.name, self.scale = int(vocab_size), int(dim), name, float(scale)
         self.norm = build_part("norm", norm) if norm is not None else None
-        self.table = None
+        self.table = self.side_table = None
+        self.side = None if side is None else (side["name"], int(side["dim"]) * int(side["layers"]))
 
     def children(self):
         return [self.norm] if self.norm is not None else []
 
     def param_specs(self):
-        return {self.name: ParamSpec((self.vocab_size, self.dim))}
+        specs = {self.name: ParamSpec((self.vocab_size, self.dim))}
+        if self.side is not None:
+            specs[self.side[0]] = ParamSpec((self.vocab_size, self.side[1]))
+        return specs
 
     def load(self, params):
         self.table = params[self.name].contiguous()
+        if self.side is not None:
+            self.side_table = params[self.side[0]].contiguous()
 
     def forward(self, ctx: StepContext) -> torch.Tensor:
         resid = torch.empty((ctx.num_tokens, self.dim), dtype=torch.float32, device=ctx.device)
         self.ops.embed(ctx.token_ids, self.table, resid, self.scale)
+        if self.side is not None:
+            ctx.step_cache[TOKEN_SIDE] = self.side_table
         if self.norm is not None:
             self.norm.norm_in_place(resid)
         return resid

@@ -13,6 +13,9 @@ gate (``act``: "relu2", the square of relu).  ``weight_on="input"``: the routing
 ``sum_e expert_e(w_e h)``, not its output (``"output"``, the default); since the first product is linear the weight is applied to
 its 32-bit sums, ahead of the activation.  ``shared_gate`` (a relative tensor name, [1, d]): the shared expert's output is
 multiplied by ``sigmoid(w_sg . h)``, one number per token; the row rides in the router's product.
+``table`` (the vocabulary's size): there is no router; an integer table ``names["table"]`` [vocab, top] gives each token id its
+experts, which weigh 1/top each (the sort below reads the table itself: no choices are written).  ``defer_combine``: the
+weighted sum is left to the block (``ExpertRows``), whose residual sum takes it in.
 
 On the device, with nothing read on the host (so a step can be captured in a graph): route -> counting sort of the
 (token, choice) pairs by expert -> grouped product gate/up over the sorted rows (rows gathered from the tokens) ->
@@ -21,6 +24,7 @@ stacked at load: ``[E, 2F, d]`` and ``[E, d, F]``.
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Dict, Optional
 
 import torch
@@ -29,13 +33,23 @@ from .base import FeedForward, ParamSpec, PartSpec, StepContext
 from ..registry import register_part, build_part
 
 
+@dataclass
+class ExpertRows:
+    """A routed feed-forward's output before its weighted sum: rows sorted by expert, where each token's stand, their common weight."""
+    rows: torch.Tensor
+    plan: dict
+    top: int
+    weight: float
+
+
 @register_part("ffn", "grouped_moe")
 class GroupedMoE(FeedForward):
     def __init__(self, prefix: str, d_model: int, hidden: int, experts: int, top: int, groups: int = 1, keep: int = 1,
                  group_top: int = 2, scale: float = 1.0, renorm: bool = False, alpha: float = 1.0,
                  limit: Optional[float] = None, shift: float = 0.0, shared: Optional[PartSpec] = None,
                  names: Optional[Dict[str, str]] = None, score: str = "sigmoid", correction: bool = False, identity: int = 0,
-                 expert: str = "glu", act: str = "relu2", weight_on: str = "output", shared_gate: Optional[str] = None):
+                 expert: str = "glu", act: str = "relu2", weight_on: str = "output", shared_gate: Optional[str] = None,
+                 table: Optional[int] = None, defer_combine: bool = False):
         super().__init__(prefix)
         if identity < 0 or experts < 0 or experts + identity < 1:
             raise ValueError(f"{experts} experts and {identity} identity experts")
@@ -58,6 +72,11 @@ class GroupedMoE(FeedForward):
             raise ValueError("a routing weight on the expert's input is built for ungated experts without identity experts")
         if shared_gate is not None and shared is None:
             raise ValueError("a gate on the shared expert needs a shared expert")
+        if table is not None and (shared is not None or identity or correction or weight_on != "output" or groups != 1 or expert != "glu"):
+            raise ValueError("experts named by a table exclude a router's options, a shared expert, identity experts and ungated experts")
+        if defer_combine and table is None:
+            raise ValueError("only experts of one common weight (named by a table) can leave their sum to the block")
+        self.vocab, self.defer_combine, self.table = None if table is None else int(table), bool(defer_combine), None
         self.expert_kind, self.act, self.weight_on_input, self.shared_gate = expert, act, weight_on == "input", shared_gate
         self.score, self.has_correction, self.identity, self.routed = score, bool(correction), int(identity), routed
         self.d_model, self.hidden, self.experts, self.top = int(d_model), int(hidden), int(experts), int(top)
@@ -65,7 +84,7 @@ class GroupedMoE(FeedForward):
         self.scale, self.renorm = float(scale), bool(renorm)
         self.alpha, self.limit, self.shift = float(alpha), limit, float(shift)
         self.shared = build_part("ffn", shared) if shared is not None else None
-        self.names = {"router": "router", "correction": "correction", "expert": "e{}", "gate": "gate", "up": "up", "down": "down"}
+        self.names = {"router": "router", "table": "table", "correction": "correction", "expert": "e{}", "gate": "gate", "up": "up", "down": "down"}
         self.correction = None
         if names:
             self.names.update(names)
@@ -78,7 +97,10 @@ class GroupedMoE(FeedForward):
 
     def param_specs(self):
         d, F = self.d_model, self.hidden
-        specs = {self.names["router"]: ParamSpec((self.routed, d), std=0.5)}
+        if self.vocab is not None:
+            specs = {self.names["table"]: ParamSpec((self.vocab, self.top), storage="table", init="distinct", high=self.experts)}
+        else:
+            specs = {self.names["router"]: ParamSpec((self.routed, d), std=0.5)}
         if self.has_correction:
             specs[self.names["correction"]] = ParamSpec((self.routed,), storage="vector", init="normal", std=0.1)
         if self.shared_gate is not None:
@@ -92,14 +114,10 @@ class GroupedMoE(FeedForward):
 
     def load(self, params):
         E = self.experts
-        self.w_router = params[self.names["router"]].contiguous()
-        if self.shared_gate is not None:                                 # the shared expert's gate: one more row of the router's product
-            self.w_router = torch.cat([self.w_router, params[self.shared_gate].reshape(1, -1)], dim=0).contiguous()
-        if self.w_router.shape[0] % 8:                                   # rows of zeros up to a multiple of 8: the library's product
-            pad = self.w_router.new_zeros((-self.w_router.shape[0] % 8, self.w_router.shape[1]))     # of many rows wants 32-byte rows of logits
-            self.w_router = torch.cat([self.w_router, pad], dim=0).contiguous()
-        if self.has_correction:
-            self.correction = params[self.names["correction"]].float().contiguous()
+        if self.vocab is not None:
+            self._load_table(params[self.names["table"]])
+        else:
+            self._load_router(params)
         if E == 0:                                                       # (identity experts only: nothing to multiply)
             self.w_gu = self.w_down = None
             return
@@ -110,6 +128,22 @@ class GroupedMoE(FeedForward):
                                      for e in range(E)]).contiguous()                    # [E, 2F, d]
         self.w_down = torch.stack([params[self._expert_name(e, "down")] for e in range(E)]).contiguous()   # [E, d, F]
 
+    def _load_table(self, table):
+        low, high = int(table.min()), int(table.max())
+        if low < 0 or high >= self.experts:
+            raise ValueError(f"{self.prefix}.{self.names['table']}: experts {low} .. {high} are named, the layer has {self.experts}")
+        self.table = table.to(torch.int32).contiguous()
+
+    def _load_router(self, params):
+        self.w_router = params[self.names["router"]].contiguous()
+        if self.shared_gate is not None:                                 # the shared expert's gate: one more row of the router's product
+            self.w_router = torch.cat([self.w_router, params[self.shared_gate].reshape(1, -1)], dim=0).contiguous()
+        if self.w_router.shape[0] % 8:                                   # rows of zeros up to a multiple of 8: the library's product
+            pad = self.w_router.new_zeros((-self.w_router.shape[0] % 8, self.w_router.shape[1]))     # of many rows wants 32-byte rows of logits
+            self.w_router = torch.cat([self.w_router, pad], dim=0).contiguous()
+        if self.has_correction:
+            self.correction = params[self.names["correction"]].float().contiguous()
+
     def validate(self, ops, dtype, page_size):
         limit = getattr(getattr(ops, "lib", None), "ttie_moe_max_experts", None)
         if limit is not None and self.routed > int(limit()):
@@ -117,6 +151,8 @@ class GroupedMoE(FeedForward):
 
     def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         ops, T = self.ops, x.shape[0]
+        if self.vocab is not None:
+            return self._table_forward(x, ctx)
         all_logits = ops.linear(x, self.w_router, None, out_dtype=torch.float32)
         logits = all_logits[:, :self.routed]
         idx, wts = ops.moe_route(logits, self.groups, self.keep, self.group_top, self.top, self.scale, self.renorm,
@@ -134,3 +170,15 @@ class GroupedMoE(FeedForward):
         gate = all_logits[:, self.routed:self.routed + 1] if self.shared_gate is not None else None
         return ops.moe_combine(y, plan, None if self.weight_on_input else wts, shared, T, self.d_model,
                                x=x if self.identity else None, shared_gate=gate)         # float32 [T, d]
+
+    def _table_forward(self, x: torch.Tensor, ctx: StepContext):
+        ops, T = self.ops, x.shape[0]
+        plan = ops.moe_plan_table(self.table, ctx.token_ids, self.experts)
+        act = ops.grouped_glu(x, self.w_gu, plan, self.top, self.hidden, self.alpha, self.limit or 0.0, self.shift)
+        y = ops.grouped_linear(act, self.w_down, plan, out_dtype=torch.float32)
+        experts = ExpertRows(y, plan, self.top, 1.0 / self.top)
+        if self.defer_combine:
+            return experts
+        out = torch.zeros((T, self.d_model), dtype=torch.float32, device=x.device)
+        ops.residual_sum(out, None, experts=(y, plan, self.top, experts.weight))
+        return out

@@ -7,7 +7,8 @@ reference fixes eps in code (models/rmsnorm.py:7) and never passes
 ``ModelConfig.rms_norm_eps``; here eps is this part's parameter.
 
 ``scalar=True``: the weight is a single number for all coordinates (a tensor of shape []); it is spread over the width when it
-is loaded, so the kernels know one form.  ``delta_norm`` (another ``RMSNorm`` of the same width): the sub-layer's output passes
+is loaded, so the kernels know one form.  ``zero_centered=True``: the stored weight is the factor less one, ``y * (1 + w)``;
+``gain``: a constant factor on the norm's result (both go into the weight in 32-bit when it is loaded).  ``delta_norm`` (another ``RMSNorm`` of the same width): the sub-layer's output passes
 that norm before it is added, in the same kernel: ``x += rms(delta) * w_d``, then ``rms(x) * w``.
 """
 from __future__ import annotations
@@ -22,19 +23,23 @@ from ..registry import register_part
 
 @register_part("norm", "rmsnorm")
 class RMSNorm(Norm):
-    def __init__(self, prefix: str, dim: int, eps: float, name: str = "weight", scalar: bool = False):
+    def __init__(self, prefix: str, dim: int, eps: float, name: str = "weight", scalar: bool = False, zero_centered: bool = False,
+                 gain: float = 1.0):
         super().__init__(prefix)
         self.dim = int(dim)
         self.eps = float(eps)
+        self.zero_centered, self.gain = bool(zero_centered), float(gain)
         self.name = name                   # relative name of the weight tensor
         self.scalar = bool(scalar)         # one number for all coordinates
         self.weight = None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
-        return {self.name: ParamSpec(() if self.scalar else (self.dim,), storage="vector", init="ones")}
+        return {self.name: ParamSpec(() if self.scalar else (self.dim,), storage="vector", init="normal" if self.zero_centered else "ones")}
 
     def load(self, params):
         w = params[self.name]
+        if self.zero_centered or self.gain != 1.0:
+            w = (w.float() + 1.0 if self.zero_centered else w.float()) * self.gain
         self.weight = w.float().expand(self.dim).contiguous() if self.scalar else w
         self._weight32 = None
 

@@ -37,15 +37,17 @@ def random_tensors(config: ModelConfig, seed: int, std: float = 0.02, perturb_no
             raise ValueError(f"tensor {name}: its shape {list(ps.shape)} leaves a size to the weight file; the configuration "
                              "must name it before random weights can be drawn")
         if ps.storage == "table":
-            # integer tables: uniform in [0, high), or 0, 1, 2, ... along the last dimension, or zeros
+            # integer tables: uniform in [0, high), or different in a row, or 0, 1, 2, ... along the last dimension, or zeros
             if ps.init == "randint" and ps.high:
                 t = torch.randint(0, int(ps.high), ps.shape, generator=gen, device=device)
+            elif ps.init == "distinct" and ps.high:                    # as many different numbers below ``high`` in every row
+                t = torch.rand((*ps.shape[:-1], int(ps.high)), generator=gen, device=device).argsort(-1)[..., :ps.shape[-1]]
             elif ps.init == "arange":
                 t = torch.arange(ps.shape[-1], device=device).expand(ps.shape)
             elif ps.init == "zeros":
                 t = torch.zeros(ps.shape, dtype=torch.int64, device=device)
             else:
-                raise ValueError(f"integer table {name}: its ParamSpec must say init='randint' (with high=), 'arange' or 'zeros'")
+                raise ValueError(f"integer table {name}: its ParamSpec must say init='randint' or 'distinct' (with high=), 'arange' or 'zeros'")
             out[name] = t.to(torch.int32).contiguous()
             continue
         if ps.init == "normal":
