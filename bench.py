@@ -367,9 +367,26 @@ def renanex_config(width, heads, layers=4):
             "layers": out, "max_seq_len": 4096}
 
 
+def fokurax_config(width, heads, layers=4):
+    """A Fokurax model at layer sizes that resemble a real model's: grouped-query attention with heads of 128 (eight query heads per
+    kv head), 64 rotated values with YaRN-rescaled frequencies, chunks of 1,024 positions; a gelu-gated feed-forward of 4 x width in
+    every fourth layer, 16 experts of width / 2, four per token, in the others; 256 side values per layer and token.  Layer
+    order: attention + dense, attention + experts, two layers on the second one's cache with experts, repeated."""
+    att = {"heads": heads, "kv_heads": max(1, heads // 8), "dim": 128, "vdim": 128, "mask": {"size": 1024}, "scale": 128 ** -0.5,
+           "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}
+    moe = {"kind": "moe", "expert": {"ff": width // 2}, "router": {"experts": 16, "top": 4}}
+    out = []
+    for i in range(layers):
+        k = i % 4
+        out.append({"type": "attention", "mixer": dict(att, kv_from=i - k + 1) if k >= 2 else dict(att),
+                    "mlp": {"kind": "dense", "ff": 4 * width} if k == 0 else moe})
+    return {"architecture": "Fokurax", "vocab": 32000, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "residual_mult": 0.7,
+            "logit_softcap": 30.0, "token_side": {"dim": 256}, "layers": out, "max_seq_len": 4096}
+
+
 DESIGNS = {"munevik": ("Munevik", munevik_config, 1024), "mizupel": ("Mizupel", mizupel_config, 1024),
            "mokalorn": ("Mokalorn", mokalorn_config, 0), "dabilorn": ("Dabilorn", dabilorn_config, 0),
-           "renanex": ("Renanex", renanex_config, 1024)}     # name, configuration, window
+           "renanex": ("Renanex", renanex_config, 1024), "fokurax": ("Fokurax", fokurax_config, 0)}     # name, configuration, window
 
 
 def like_config(width, heads, layers=4):
@@ -386,7 +403,8 @@ class OpRecorder:
              "rglru_scan", "glu", "linear_glu", "grouped_glu", "moe_route", "moe_plan", "grouped_linear", "moe_combine",
              "qkv_conv_rope_store", "conv_tail_update", "gate_head_rows", "token_shift_mix", "wkv_scan", "mlstm_scan", "head_norm_gate",
              "activation", "linear_act", "wkv_decay", "mlstm_gates", "rotate_heads", "retention_scan", "stream_conv", "proj_row_rms",
-             "rmsnorm_cols", "grouped_act", "sandwich_norm", "joint_qkv_store", "paged_attention_joint", "selective_scan", "activation_rows", "linear_narrow")
+             "rmsnorm_cols", "grouped_act", "sandwich_norm", "joint_qkv_store", "paged_attention_joint", "selective_scan", "activation_rows", "linear_narrow",
+             "residual_sum", "token_gate", "moe_plan_table")
 
     def __init__(self, ops):
         self.ops, self.calls, self.orig, self.depth = ops, [], {}, 0
@@ -454,6 +472,13 @@ def op_cost(name, args, kw, out, kv_lens, window):
         rows = kw.get("num_rows") or args[0].shape[0]
         per = args[0].shape[1] * ((4 if kw.get("rows") is not None else 8) + args[6].element_size())
         return rows * per + _tensor_bytes(args[1]) * rows // args[0].shape[0], 0
+    if name == "residual_sum":                                     # (resid, a, f): the stream read and written, every term read, the copy written
+        ex = kw.get("experts")
+        return 2 * _tensor_bytes(args[0]) + _tensor_bytes(list(args[1:3])) + _tensor_bytes([ex[0], ex[1]["pos_of_pair"]] if ex else []) + _tensor_bytes(out), 0
+    if name == "token_gate":                                       # (z, ids, table, col0, n, ...): of the table one layer's values per token
+        return _tensor_bytes([args[0], args[1], out]) + args[1].shape[0] * args[4] * args[2].element_size(), 0
+    if name == "moe_plan_table":                                   # (table, ids, ...): a row of the table per token
+        return args[1].shape[0] * (1 + args[0].shape[1]) * 4 + _tensor_bytes(out), 0
     if name == "activation_rows":                                  # (x, cols, ...)
         return args[0].shape[0] * args[1] * args[0].element_size() + _tensor_bytes(out), 0
     if name == "joint_qkv_store":                                  # the projected row read, joint query rows written, joint key and value rows stored
@@ -628,8 +653,8 @@ def run_design(args, pk):
 
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default=None, choices=("munevik", "mizupel", "mokalorn", "dabilorn", "renanex"), help="prefill and decode of this design at a few sizes beside the closest existing model, with per-operation times")
-    ap.add_argument("--beside", default=None, choices=("mqa_gpt", "munevik", "mizupel", "mokalorn", "dabilorn", "renanex"), help="with --design: the model it is timed beside (default: the multi-query GPT)")
+    ap.add_argument("--design", default=None, choices=("munevik", "mizupel", "mokalorn", "dabilorn", "renanex", "fokurax"), help="prefill and decode of this design at a few sizes beside the closest existing model, with per-operation times")
+    ap.add_argument("--beside", default=None, choices=("mqa_gpt", "munevik", "mizupel", "mokalorn", "dabilorn", "renanex", "fokurax"), help="with --design: the model it is timed beside (default: the multi-query GPT)")
     ap.add_argument("--sizes", default=None, help="with --design: comma-separated model widths (multiples of 128)")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=64)
