@@ -477,8 +477,8 @@ def op_cost(name, args, kw, out, kv_lens, window):
         return 2 * _tensor_bytes(args[0]) + _tensor_bytes(list(args[1:3])) + _tensor_bytes([ex[0], ex[1]["pos_of_pair"]] if ex else []) + _tensor_bytes(out), 0
     if name == "token_gate":                                       # (z, ids, table, col0, n, ...): of the table one layer's values per token
         return _tensor_bytes([args[0], args[1], out]) + args[1].shape[0] * args[4] * args[2].element_size(), 0
-    if name == "moe_plan_table":                                   # (table, ids, ...): a row of the table per token
-        return args[1].shape[0] * (1 + args[0].shape[1]) * 4 + _tensor_bytes(out), 0
+    if name == "moe_plan_table":                                   # (tables, ids, ...): a row of every layer's table per token
+        return args[1].shape[0] * (1 + args[0].shape[0] * args[0].shape[2]) * 4 + _tensor_bytes(out), 0
     if name == "activation_rows":                                  # (x, cols, ...)
         return args[0].shape[0] * args[1] * args[0].element_size() + _tensor_bytes(out), 0
     if name == "joint_qkv_store":                                  # the projected row read, joint query rows written, joint key and value rows stored

@@ -466,32 +466,32 @@ def test_table_experts_alone(ops, dtype, T, experts, top):
         assert rel(y, pf.table_experts(x.double(), w, "", f, toks)) < (2e-5 if dtype == "float32" else 2e-2)
 
 
-@pytest.mark.parametrize("P", [1, 63, 700])
-def test_plan_from_a_table(ops, P):
-    """Every pair stands once among its expert's rows; the row tiles cover each expert's rows once."""
+@pytest.mark.parametrize("T", [1, 63, 700])
+def test_plans_from_tables(ops, T):
+    """Three layers' plans in one launch: every pair stands once among its expert's rows; the row tiles cover each expert's rows once."""
     vocab, top, E = 50, 3, 11
-    g = torch.Generator().manual_seed(P)
-    table = torch.rand(vocab, E, generator=g).argsort(-1)[:, :top].to(torch.int32)
-    ids = torch.randint(0, vocab, (P,), generator=g).to(torch.int32)
-    plan = ops.moe_plan_table(table.to(DEV), ids.to(DEV), E)
-    want = table[ids.long()].reshape(-1)
-    offs, pos, pair = plan["offsets"].cpu(), plan["pos_of_pair"].cpu(), plan["pair_of_pos"].cpu()
-    assert offs.tolist() == [0] + torch.bincount(want, minlength=E).cumsum(0).tolist()
-    assert torch.equal(pair[pos.long()], torch.arange(P * top, dtype=torch.int32))
-    assert all(offs[e] <= pos[i] < offs[e + 1] for i, e in enumerate(want.tolist()))
-    covered = torch.zeros(P * top, dtype=torch.int64)
-    for e, first, rows, _ in plan["tiles"].view(-1, 4)[:int(plan["meta"][0])].tolist():
-        assert offs[e] <= first and first + rows <= offs[e + 1] and 0 < rows
-        covered[first:first + rows] += 1
-    assert (covered == 1).all()
+    g = torch.Generator().manual_seed(T)
+    tables = torch.rand(3, vocab, E, generator=g).argsort(-1)[..., :top].to(torch.int32)
+    ids = torch.randint(0, vocab, (T,), generator=g).to(torch.int32)
+    for table, plan in zip(tables, ops.moe_plan_table(tables.to(DEV), ids.to(DEV), E)):
+        want = table[ids.long()].reshape(-1)
+        offs, pos, pair = plan["offsets"].cpu(), plan["pos_of_pair"].cpu(), plan["pair_of_pos"].cpu()
+        assert offs.tolist() == [0] + torch.bincount(want, minlength=E).cumsum(0).tolist()
+        assert torch.equal(pair[pos.long()], torch.arange(T * top, dtype=torch.int32))
+        assert all(offs[e] <= pos[i] < offs[e + 1] for i, e in enumerate(want.tolist()))
+        covered = torch.zeros(T * top, dtype=torch.int64)
+        for e, first, rows, _ in plan["tiles"].view(-1, 4)[:int(plan["meta"][0])].tolist():
+            assert offs[e] <= first and first + rows <= offs[e + 1] and 0 < rows
+            covered[first:first + rows] += 1
+        assert (covered == 1).all()
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("d", [64, 50, 1032])
+@pytest.mark.parametrize("T,d", [(9, 64), (9, 50), (9, 1032), (1030, 1032), (600, 1748)])
 @pytest.mark.parametrize("kind", ["rows", "parts", "experts", "alone"])
-def test_residual_sum(ops, dtype, d, kind):
+def test_residual_sum(ops, dtype, T, d, kind):
     """x + mult * (a + f + bias) with f as rows, as partial sums, as sorted expert rows (either dtype), or absent."""
-    T, top = 9, 3
+    top = 3
     g = torch.Generator().manual_seed(d)
     r = lambda *s: torch.randn(s, generator=g)
     resid, bias = r(T, d), r(d)
@@ -517,7 +517,7 @@ def test_residual_sum(ops, dtype, d, kind):
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("T", [1, 6, 33, 200])
-@pytest.mark.parametrize("width,dim,layer_index", [(72, 1, 0), (72, 10, 2), (50, 13, 1), (512, 64, 1)])
+@pytest.mark.parametrize("width,dim,layer_index", [(72, 1, 0), (72, 10, 2), (50, 13, 1), (512, 64, 1), (48, 8, 2)])
 def test_side_input_alone(ops, dtype, T, width, dim, layer_index):
     """The layer's own columns of the token's row; the matrices' padding adds nothing."""
     vocab, layers = 29, 3

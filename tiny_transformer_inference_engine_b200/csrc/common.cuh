@@ -119,6 +119,9 @@ int num_sms();
 // kernels here call it first thing, so only launch latency and CTA scheduling overlap).  Works inside
 // captured graphs.  ttie_set_pdl(0) turns it off.
 bool pdl_enabled();
+// asks (and clears) whether the next kernel is to be launched as an ordinary one although pdl_enabled(): the first kernel of a stream
+// behind a wait for another stream's event
+bool pdl_skip_once();
 // cluster: CTAs per thread-block cluster along x, y, z (the grid must be a multiple); dim3(1) for none.
 template <typename... KArgs, typename... Args>
 inline cudaError_t launch_kernel(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t s, dim3 cluster,
@@ -129,7 +132,7 @@ inline cudaError_t launch_kernel(void (*kernel)(KArgs...), dim3 grid, dim3 block
     int n = 0;
     // (a cluster launch does not take the attribute: as a programmatic dependent it was measured to start late)
     const bool clustered = cluster.x * cluster.y * cluster.z > 1;
-    if (pdl_enabled() && !clustered) {
+    if (!pdl_skip_once() && pdl_enabled() && !clustered) {
         attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
         attr[n].val.programmaticStreamSerializationAllowed = 1;
         ++n;

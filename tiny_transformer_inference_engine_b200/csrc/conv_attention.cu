@@ -201,11 +201,12 @@ __device__ __forceinline__ float head_sum(float v, int lanes) {
 __global__ void __launch_bounds__(256) qkv_conv_rope_store_vec8_kernel(const QkvArgs a, int T_) {
     TTIE_PDL_ENTRY();
     const int chunks = a.Dp >> 3, units = a.Hq + 2 * a.Hkv;
-    const long long id = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (id >= (long long)T_ * units * chunks) return;
-    const int jc = (int)(id % chunks);
-    const int unit = (int)((id / chunks) % units);
-    const int t = (int)(id / ((long long)chunks * units));
+    const unsigned id = blockIdx.x * blockDim.x + threadIdx.x;       // (the caller keeps the count of threads below 2^31)
+    if (id >= (unsigned)T_ * units * chunks) return;
+    const unsigned head = id / (unsigned)chunks;
+    const int jc = (int)(id - head * chunks);
+    const int t = (int)(head / (unsigned)units);
+    const int unit = (int)(head - (unsigned)t * units);
     const int C = row_channels(a);
     const int kind = unit < a.Hq ? 0 : unit < a.Hq + a.Hkv ? 1 : 2;
     const int h = kind == 0 ? unit : kind == 1 ? unit - a.Hq : unit - a.Hq - a.Hkv;
@@ -256,16 +257,18 @@ __global__ void __launch_bounds__(256) qkv_conv_rope_store_vec8_kernel(const Qkv
             }
             const int f0 = low ? i0 : i0 - half;
 #pragma unroll
-            for (int i = 0; i < 8; ++i) {
-                const float2 c = cs[f0 + i];
+            for (int i = 0; i < 8; i += 2) {                         // (two pairs' cos and sin per load: f0 and the row are multiples of 4 pairs)
+                const float4 c = __ldg(reinterpret_cast<const float4*>(cs + f0 + i));
                 out[i] = low ? out[i] * c.x - other[i] * c.y : out[i] * c.x + other[i] * c.y;
+                out[i + 1] = low ? out[i + 1] * c.z - other[i + 1] * c.w : out[i + 1] * c.z + other[i + 1] * c.w;
             }
         } else {
 #pragma unroll
-            for (int i = 0; i < 8; i += 2) {
-                const float2 c = cs[(i0 + i) >> 1];
-                const float x = out[i], y = out[i + 1];
+            for (int i = 0; i < 8; i += 4) {
+                const float4 c = __ldg(reinterpret_cast<const float4*>(cs + ((i0 + i) >> 1)));
+                const float x = out[i], y = out[i + 1], z = out[i + 2], w = out[i + 3];
                 out[i] = x * c.x - y * c.y; out[i + 1] = x * c.y + y * c.x;
+                out[i + 2] = z * c.z - w * c.w; out[i + 3] = z * c.w + w * c.z;
             }
         }
     }
@@ -480,9 +483,8 @@ extern "C" int ttie_qkv_conv_rope_store(const void* proj, long long ld, int T, i
     const int lanes = Dp / 8;                                        // of a head in the eight-values form; a norm adds up over them by shuffles
     const bool norm_ok = ((!norm_w || row_inv) && after_eps < 0.f) || (Dp % 8 == 0 && lanes <= 32 && (lanes & (lanes - 1)) == 0);
     if (dtype == kBF16 && D % 8 == 0 && Dv % 8 == 0 && Dp % 8 == 0 && ld % 8 == 0 && aligned && norm_ok
-        && (rot == 0 || rot % (style == 1 ? 16 : 8) == 0)) {
+        && (rot == 0 || (rot % (style == 1 ? 16 : 8) == 0 && !((uintptr_t)cs & 15))) && (long long)T * (Hq + 2 * Hkv) * (Dp / 8) < (1LL << 31)) {
         const long long threads = (long long)T * (Hq + 2 * Hkv) * (Dp / 8);
-        if ((threads + 255) / 256 > 2147483647LL) TTIE_FAIL("qkv_conv_rope_store: grid too large");
         TTIE_LAUNCH(qkv_conv_rope_store_vec8_kernel, (unsigned)((threads + 255) / 256), 256, 0, s, a, T);
         TTIE_CHECK_LAUNCH("qkv_conv_rope_store");
         return 0;

@@ -28,6 +28,11 @@ bool pdl_enabled() {
 }
 }  // namespace ttie
 extern "C" void ttie_set_pdl(int on) { ttie::g_pdl = on ? 1 : 0; }
+namespace ttie {
+static thread_local bool g_pdl_skip = false;
+bool pdl_skip_once() { const bool skip = g_pdl_skip; g_pdl_skip = false; return skip; }
+}  // namespace ttie
+extern "C" int ttie_pdl_skip_once() { ttie::g_pdl_skip = true; return 0; }
 
 namespace ttie {
 int num_sms() {

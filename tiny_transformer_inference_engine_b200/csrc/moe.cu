@@ -34,12 +34,12 @@ __global__ void glu_kernel(const T* __restrict__ gu, long long ld, T* __restrict
 }
 
 // bfloat16, 8 values per thread (F and the row stride multiples of 8, 16-byte aligned rows)
-__global__ void glu_vec8_kernel(const __nv_bfloat16* __restrict__ gu, long long ld, __nv_bfloat16* __restrict__ out, int F8, size_t total8,
+__global__ void __launch_bounds__(128) glu_vec8_kernel(const __nv_bfloat16* __restrict__ gu, long long ld, __nv_bfloat16* __restrict__ out, int F8, int T_,
                                 float alpha, float limit, float shift, int act) {
     TTIE_PDL_ENTRY();
-    for (size_t e = blockIdx.x * (size_t)blockDim.x + threadIdx.x; e < total8; e += (size_t)gridDim.x * blockDim.x) {
-        const size_t t = e / F8;
-        const int f = (int)(e % F8) * 8;
+    const int f = (blockIdx.x * blockDim.x + threadIdx.x) * 8;       // grid: (columns, rows)
+    if (f >= F8 * 8) return;
+    for (size_t t = blockIdx.y; t < (size_t)T_; t += gridDim.y) {
         const uint4 gv = *reinterpret_cast<const uint4*>(gu + t * ld + f);
         const uint4 uv = *reinterpret_cast<const uint4*>(gu + t * ld + (size_t)F8 * 8 + f);
         const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv);
@@ -132,20 +132,23 @@ moe_route_kernel(const float* __restrict__ logits, long long ld, int T_, int E, 
     for (int k = lane; k < top; k += 32) wts[(size_t)t * top + k] *= renorm ? scale / total : scale;
 }
 
-// one CTA.  pairs P = T * top.  tiles: int32 [max_tiles][4] = (expert, first row, rows, 0); meta[0] = number of tiles.
-// `table` (int32 [vocab][top], optional): there are no router's choices; the row of a token's id lists its experts.  Otherwise idx[p].
+// One CTA per layer.  pairs P = T * top.  tiles: int32 [max_tiles][4] = (expert, first row, rows, 0); meta[0] = number of tiles.
+// `table` (int32 [layers][vocab][top], optional): there are no router's choices; the row of a token's id lists its experts, so every
+// layer's plan can be made at once (outputs `out_stride` ints apart).  Otherwise idx[p], one layer.
 struct Choices { const int* idx; const int* table; const int* token_ids; int top, vocab, E; };
 __device__ __forceinline__ int expert_of(const Choices& c, int p) {
     if (!c.table) return c.idx[p];
     const int t = p / c.top;
     const int id = min(max(c.token_ids[t], 0), c.vocab - 1);        // ids and entries are validated on the host; never count outside
-    return min(max(c.table[(size_t)id * c.top + (p - t * c.top)], 0), c.E - 1);
+    return min(max(__ldg(c.table + ((size_t)blockIdx.x * c.vocab + id) * c.top + (p - t * c.top)), 0), c.E - 1);
 }
 __global__ void __launch_bounds__(1024)
 moe_plan_kernel(const Choices ch, int P, int E, int tile_experts, int tile_rows, int max_tiles, int* __restrict__ offsets,
-                int* __restrict__ pos_of_pair, int* __restrict__ pair_of_pos, int* __restrict__ tiles, int* __restrict__ meta) {
+                int* __restrict__ pos_of_pair, int* __restrict__ pair_of_pos, int* __restrict__ tiles, int* __restrict__ meta, long long out_stride) {
     __shared__ int count[MAX_EXPERTS], cursor[MAX_EXPERTS];
     TTIE_PDL_ENTRY();
+    const long long at_layer = blockIdx.x * out_stride;
+    offsets += at_layer; pos_of_pair += at_layer; pair_of_pos += at_layer; tiles += at_layer; meta += at_layer;
     for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
     __syncthreads();
     for (int p = threadIdx.x; p < P; p += blockDim.x) atomicAdd(&count[expert_of(ch, p)], 1);
@@ -368,6 +371,22 @@ __global__ void gather_rows_kernel(const T* __restrict__ x, long long ldx, const
     }
 }
 
+// the same in pieces of 16 bytes (a row and the strides hold whole ones): `per` pieces a row, ld pieces from row to row of x
+__global__ void __launch_bounds__(128) gather_rows_16b_kernel(const uint4* __restrict__ x, long long ld, const int* __restrict__ row_of, int row_div,
+                                                              int rows, int per, uint4* __restrict__ out) {
+    TTIE_PDL_ENTRY();
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;             // grid: (pieces, tiles of GATHER_ROWS rows)
+    if (i >= per) return;
+    constexpr int GATHER_ROWS = 4;                                   // loads in flight per thread
+    for (int r0 = blockIdx.y * GATHER_ROWS; r0 < rows; r0 += gridDim.y * GATHER_ROWS) {
+        uint4 v[GATHER_ROWS];
+#pragma unroll
+        for (int k = 0; k < GATHER_ROWS; ++k) if (r0 + k < rows) v[k] = __ldg(x + (size_t)(row_of[r0 + k] / row_div) * ld + i);
+#pragma unroll
+        for (int k = 0; k < GATHER_ROWS; ++k) if (r0 + k < rows) out[(size_t)(r0 + k) * per + i] = v[k];
+    }
+}
+
 template <typename T, typename TY>
 __global__ void moe_combine_kernel(const TY* __restrict__ Y, const int* __restrict__ pos_of_pair, const float* __restrict__ wts,
                                    const T* __restrict__ shared, int T_, int d, int top, float* __restrict__ out,
@@ -431,8 +450,8 @@ extern "C" int ttie_glu(const void* gate_up, long long ld, void* out, int T, int
     if (act < 0 || act > 1) TTIE_FAIL("glu: unknown activation %d", act);
     const size_t total = (size_t)T * F;
     if (dtype == kBF16 && F % 8 == 0 && ld % 8 == 0 && (((uintptr_t)gate_up | (uintptr_t)out) & 15) == 0) {
-        TTIE_LAUNCH(glu_vec8_kernel, grid_for(total / 8), 256, 0, (cudaStream_t)stream, (const __nv_bfloat16*)gate_up, ld, (__nv_bfloat16*)out, F / 8,
-                    total / 8, alpha, limit, shift, act);
+        TTIE_LAUNCH(glu_vec8_kernel, dim3(ceil_div(F / 8, 128), T < 65535 ? T : 65535), 128, 0, (cudaStream_t)stream, (const __nv_bfloat16*)gate_up, ld,
+                    (__nv_bfloat16*)out, F / 8, T, alpha, limit, shift, act);
         TTIE_CHECK_LAUNCH("glu");
         return 0;
     }
@@ -457,24 +476,26 @@ extern "C" int ttie_moe_route(const float* logits, long long ld, int T, int E, i
     return 0;
 }
 
-static int launch_plan(const Choices& ch, int P, int E, int tile_experts, int max_tiles, int* offsets, int* pos_of_pair, int* pair_of_pos,
+static int launch_plan(const Choices& ch, int layers, long long out_stride, int P, int E, int tile_experts, int max_tiles, int* offsets, int* pos_of_pair, int* pair_of_pos,
                        int* tiles, int* meta, cudaStream_t s) {
     if (P <= 0) return 0;
     if (E > MAX_EXPERTS) TTIE_FAIL("moe_plan: %d experts (limit %d)", E, MAX_EXPERTS);
     if (tile_experts < 0 || tile_experts > E) TTIE_FAIL("moe_plan: %d of %d experts own matrices", tile_experts, E);
-    TTIE_LAUNCH(moe_plan_kernel, 1, 1024, 0, s, ch, P, E, tile_experts, BM, max_tiles, offsets, pos_of_pair, pair_of_pos, tiles, meta);
+    TTIE_LAUNCH(moe_plan_kernel, layers, 1024, 0, s, ch, P, E, tile_experts, BM, max_tiles, offsets, pos_of_pair, pair_of_pos, tiles, meta, out_stride);
     TTIE_CHECK_LAUNCH("moe_plan");
     return 0;
 }
 extern "C" int ttie_moe_plan(const int* idx, int P, int E, int tile_experts, int max_tiles, int* offsets, int* pos_of_pair, int* pair_of_pos,
                              int* tiles, int* meta, void* stream) {
-    return launch_plan({idx, nullptr, nullptr, 1, 1, E}, P, E, tile_experts, max_tiles, offsets, pos_of_pair, pair_of_pos, tiles, meta, (cudaStream_t)stream);
+    return launch_plan({idx, nullptr, nullptr, 1, 1, E}, 1, 0, P, E, tile_experts, max_tiles, offsets, pos_of_pair, pair_of_pos, tiles, meta, (cudaStream_t)stream);
 }
-// the experts come from a table of the token ids: table int32 [vocab][top], token_ids int32 [T]
-extern "C" int ttie_moe_plan_table(const int* table, int vocab, const int* token_ids, int T, int top, int E, int max_tiles, int* offsets,
-                                   int* pos_of_pair, int* pair_of_pos, int* tiles, int* meta, void* stream) {
+// the experts come from a table of the token ids: table int32 [layers][vocab][top], token_ids int32 [T]; the outputs are the first
+// layer's, each next layer's lie out_stride ints further
+extern "C" int ttie_moe_plan_table(const int* table, int layers, long long out_stride, int vocab, const int* token_ids, int T, int top, int E,
+                                   int max_tiles, int* offsets, int* pos_of_pair, int* pair_of_pos, int* tiles, int* meta, void* stream) {
+    if (layers < 1) return 0;
     if (top < 1 || top > E || vocab < 1) TTIE_FAIL("moe_plan: a table of %d rows with %d of %d experts", vocab, top, E);
-    return launch_plan({nullptr, table, token_ids, top, vocab, E}, T * top, E, E, max_tiles, offsets, pos_of_pair, pair_of_pos, tiles, meta, (cudaStream_t)stream);
+    return launch_plan({nullptr, table, token_ids, top, vocab, E}, layers, out_stride, T * top, E, E, max_tiles, offsets, pos_of_pair, pair_of_pos, tiles, meta, (cudaStream_t)stream);
 }
 
 // act, row_scale, scale_of: an activation behind an ungated product, see RowAct (act 0 and row_scale null: the plain product)
@@ -532,6 +553,14 @@ extern "C" int ttie_grouped_gemm_act(const void* A, long long lda, const int* ro
 extern "C" int ttie_gather_rows(const void* x, long long ldx, const int* row_of, int row_div, int rows, int d, void* out, int dtype, void* stream) {
     if (rows <= 0) return 0;
     const size_t total = (size_t)rows * d;
+    const int vn = dtype == kF32 ? 4 : 8;                            // values in 16 bytes
+    if (d % vn == 0 && ldx % vn == 0 && !(((uintptr_t)x | (uintptr_t)out) & 15)) {
+        const int tiles = ceil_div(rows, 4);
+        TTIE_LAUNCH(gather_rows_16b_kernel, dim3(ceil_div(d / vn, 128), tiles < 65535 ? tiles : 65535), 128, 0, (cudaStream_t)stream, (const uint4*)x, ldx / vn,
+                    row_of, row_div > 0 ? row_div : 1, rows, d / vn, (uint4*)out);
+        TTIE_CHECK_LAUNCH("gather_rows");
+        return 0;
+    }
     if (dtype == kF32) TTIE_LAUNCH(gather_rows_kernel<float>, grid_for(total), 256, 0, (cudaStream_t)stream, (const float*)x, ldx, row_of, row_div > 0 ? row_div : 1, rows, d, (float*)out);
     else TTIE_LAUNCH(gather_rows_kernel<__nv_bfloat16>, grid_for(total), 256, 0, (cudaStream_t)stream, (const __nv_bfloat16*)x, ldx, row_of, row_div > 0 ? row_div : 1, rows, d, (__nv_bfloat16*)out);
     TTIE_CHECK_LAUNCH("gather_rows");

@@ -69,6 +69,9 @@ class Model:
             owners[pid].load(params)
         if getattr(self.head, "tied_to_embedding", False):
             self.head.tie(self.embedding)
+        parts = self.parts()
+        for p in parts:
+            p.link(parts)
         tune = getattr(getattr(self, "ops", None), "tune_products", None)
         if tune is not None:                                       # the kernel library may measure which product suits each shape
             tune([w for p in self.parts() for w in p.product_weights() if w is not None])

@@ -12,6 +12,7 @@ reduced-precision matrix mode can slip in.
 """
 from __future__ import annotations
 
+import contextlib
 import ctypes
 import math
 import os
@@ -97,11 +98,12 @@ _SIGNATURES = {
                         _c_int, _c_void, _c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void, _c_int, _c_void,
                         _c_int, _c_void],
     "ttie_glu": [_c_void, _c_ll, _c_void, _c_int, _c_int, _c_float, _c_float, _c_float, _c_int, _c_int, _c_void],
+    "ttie_pdl_skip_once": [],
     "ttie_residual_sum": [_c_void, _c_void, _c_void, _c_int, _c_ll, _c_void, _c_void, _c_int, _c_ll, _c_void, _c_int, _c_void, _c_int, _c_float,
                           _c_void, _c_float, _c_void, _c_int, _c_int, _c_int, _c_void],
     "ttie_token_gate": [_c_void, _c_void, _c_int, _c_ll, _c_void, _c_void, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int, _c_void],
     "ttie_moe_route": [_c_void, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void, _c_void, _c_void, _c_void],
-    "ttie_moe_plan_table": [_c_void, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void],
+    "ttie_moe_plan_table": [_c_void, _c_int, _c_ll, _c_int, _c_void, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void],
     "ttie_moe_plan": [_c_void, _c_int, _c_int, _c_int, _c_int, _c_void, _c_void, _c_void, _c_void, _c_void, _c_void],
     "ttie_grouped_gemm": [_c_void, _c_ll, _c_void, _c_int, _c_void, _c_ll, _c_ll, _c_void, _c_ll, _c_void, _c_void, _c_int, _c_int, _c_int,
                           _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float, _c_void],
@@ -170,6 +172,7 @@ class CudaOps:
             fn = getattr(self.lib, name)
             fn.argtypes, fn.restype = argtypes, _c_int
         self.lib.ttie_last_error.restype = ctypes.c_char_p
+        self._branch = None                   # (second stream, event at the fork, event at its end), made when first used
         self.launches = 0                     # kernels of this library launched so far
         self.num_sms = int(torch.cuda.get_device_properties(self.device).multi_processor_count)   # the plans below are sized for it
         self._device_index = self.device.index if self.device.index is not None else torch.cuda.current_device()
@@ -1413,6 +1416,29 @@ class CudaOps:
         return out
 
     # ---- sub-layers in parallel, a token's own input
+    branch_max_tokens = 64                  # tokens of a step up to which independent sub-layers run on two streams
+
+    @contextlib.contextmanager
+    def branch(self):
+        """Launches inside the block go to a second stream, behind everything launched so far; ``join`` makes the current stream wait
+        for them.  Works while a graph is captured (its two branches then run side by side in a replay).  What the block
+        allocates belongs to the second stream: the next ``branch`` starts behind every use of it before that point, so memory is
+        handed on in order."""
+        main = torch.cuda.current_stream(self.device)
+        if self._branch is None:
+            self._branch = (torch.cuda.Stream(self.device), torch.cuda.Event(), torch.cuda.Event())
+        side, fork, done = self._branch
+        fork.record(main)
+        side.wait_event(fork)
+        self.lib.ttie_pdl_skip_once()
+        with torch.cuda.stream(side):
+            yield
+            done.record(side)
+
+    def join(self):
+        torch.cuda.current_stream(self.device).wait_event(self._branch[2])
+        self.lib.ttie_pdl_skip_once()
+
     def residual_sum(self, resid, a, f=None, experts=None, bias=None, mult=1.0, out_dtype=None):
         """resid <- resid + mult * (a + f + bias) over the 32-bit stream [T, d], in one pass.  ``a``, ``f`` (or None): sub-layers'
         outputs, [T, d] in the compute dtype or float32, or float32 partial sums [S, T, d]; ``experts`` (rows [P, d], plan, top,
@@ -1520,23 +1546,28 @@ class CudaOps:
         self.launches += 1
         return plan
 
-    def moe_plan_table(self, table, token_ids, num_experts):
-        """``moe_plan`` for experts that a table names: row ``token_ids[t]`` of ``table`` (int32 [vocab, top]) lists token t's
-        experts.  One launch; no choices are written (the plan's ``idx`` is None)."""
-        T, (vocab, top) = token_ids.shape[0], table.shape
+    def moe_plan_table(self, tables, token_ids, num_experts):
+        """``moe_plan`` for experts that tables name: row ``token_ids[t]`` of layer l's table (``tables`` int32 [layers, vocab, top])
+        lists token t's experts in that layer.  The plans of all layers in one launch, a list; no choices are written (a plan's
+        ``idx`` is None)."""
+        T, (layers, vocab, top) = token_ids.shape[0], tables.shape
         P = T * top
         max_tiles = P // int(self.lib.ttie_moe_tile_rows()) + num_experts
-        buf = torch.empty(2 * P + num_experts + 1 + 4 * max_tiles + 4, dtype=torch.int32, device=token_ids.device)
-        plan = {"pos_of_pair": buf[:P], "pair_of_pos": buf[P:2 * P], "offsets": buf[2 * P:2 * P + num_experts + 1],
-                "tiles": buf[2 * P + num_experts + 1:2 * P + num_experts + 1 + 4 * max_tiles], "meta": buf[-4:], "max_tiles": max_tiles,
-                "pairs": P, "idx": None, "real_experts": num_experts}
-        self._check(self.lib.ttie_moe_plan_table(_ptr(table), vocab, _ptr(token_ids), T, top, num_experts, max_tiles, _ptr(plan["offsets"]),
-                                                 _ptr(plan["pos_of_pair"]), _ptr(plan["pair_of_pos"]), _ptr(plan["tiles"]), _ptr(plan["meta"]),
-                                                 self._stream(token_ids)), "moe_plan_table")
+        o = [0, P, 2 * P, 2 * P + num_experts + 1]                                # pos_of_pair, pair_of_pos, offsets, tiles, meta
+        o.append(o[3] + 4 * max_tiles)
+        size = (o[4] + 4 + 3) & ~3
+        buf = torch.empty((layers, size), dtype=torch.int32, device=token_ids.device)
+        plans = [{"pos_of_pair": b[:P], "pair_of_pos": b[P:2 * P], "offsets": b[o[2]:o[3]], "tiles": b[o[3]:o[4]], "meta": b[o[4]:o[4] + 4],
+                  "max_tiles": max_tiles, "pairs": P, "idx": None, "real_experts": num_experts} for b in buf.unbind(0)]
+        first = plans[0]
+        self._check(self.lib.ttie_moe_plan_table(_ptr(tables), layers, size, vocab, _ptr(token_ids), T, top, num_experts, max_tiles,
+                                                 _ptr(first["offsets"]), _ptr(first["pos_of_pair"]), _ptr(first["pair_of_pos"]), _ptr(first["tiles"]),
+                                                 _ptr(first["meta"]), self._stream(token_ids)), "moe_plan_table")
         self.launches += 1
-        return plan
+        return plans
 
-    grouped_few_rows = 64                   # (token, choice) pairs up to which the grouped product streams every tile's weights once
+    grouped_few_rows = 48                   # (token, choice) pairs up to which the grouped product streams every tile's weights once (16 experts of [1024, 1024] to
+                                            # [4096, 4096]: ahead of the library up to 32 to 48 pairs, level or behind at 64)
 
     def _library_grouped(self, x, w, plan, gather_div):
         """The library's grouped product (bfloat16, many rows): rows gathered into expert order, then one call whose group

@@ -216,6 +216,9 @@ class Part:
         """Receives this part's tensors (relative names), already on the device and in
         the storage class its ParamSpec asked for."""
 
+    def link(self, parts: List["Part"]) -> None:
+        """Called once all parts of the model (``parts``, in layer order) are loaded: a part may join what it keeps with others'."""
+
     def bind(self, ops, dtype: torch.dtype, device: torch.device) -> None:
         self.ops, self.dtype, self.device = ops, dtype, device
         for c in self.children():

@@ -187,6 +187,8 @@ class ParallelBlock(Block):
     """One norm, whose output both sub-layers read, and one sum: ``x = x + mult * (mixer(h) + ffn(h))`` with ``h = norm(x)``; a layer
     without a feed-forward (``ffn`` None) adds the mixer's output alone.  One kernel forms the sum: it takes the sub-layers'
     outputs as they leave their last products (partial sums, rows sorted by expert, a bias that the feed-forward left to the block).
+    Neither sub-layer waits for the other: in steps of a few tokens they run on two streams, so that the feed-forward's weights
+    stream in beside attention's latencies.
 
     ``side`` and ``side_norm`` (None: neither): a third sub-layer behind that sum which reads the stream itself,
     ``x = x + side_norm(side(x))``; ``mult`` on it is the norm part's ``gain``.  Its output waits unnormed in ``stream.delta`` with the
@@ -214,8 +216,16 @@ class ParallelBlock(Block):
         ops, resid = self.ops, stream.resid
         pending = {} if stream.delta_norm is None else {"delta_norm": stream.delta_norm}
         h = self.norm.add_norm(resid, stream.delta, **pending)
+        f = None
+        apart = self.ffn is not None and ctx.num_tokens <= getattr(ops, "branch_max_tokens", 0)
+        if apart:
+            with ops.branch():
+                f = self.ffn.forward(h, ctx)
         a = self.mixer.forward(h, ctx, mixer_cache_argument(self.mixer, caches))
-        f = self.ffn.forward(h, ctx) if self.ffn is not None else None
+        if apart:
+            ops.join()
+        elif self.ffn is not None:
+            f = self.ffn.forward(h, ctx)
         experts = (f.rows, f.plan, f.top, f.weight) if isinstance(f, ExpertRows) else None
         narrow = self.side is not None and self.dtype != resid.dtype         # the side sub-layer reads the stream in the compute dtype
         x = ops.residual_sum(resid, a, None if experts is not None else f, experts=experts, bias=getattr(self.ffn, "out_bias", None),

@@ -14,7 +14,8 @@ gate (``act``: "relu2", the square of relu).  ``weight_on="input"``: the routing
 its 32-bit sums, ahead of the activation.  ``shared_gate`` (a relative tensor name, [1, d]): the shared expert's output is
 multiplied by ``sigmoid(w_sg . h)``, one number per token; the row rides in the router's product.
 ``table`` (the vocabulary's size): there is no router; an integer table ``names["table"]`` [vocab, top] gives each token id its
-experts, which weigh 1/top each (the sort below reads the table itself: no choices are written).  ``defer_combine``: the
+experts, which weigh 1/top each.  The sort below reads the tables itself (no choices are written) and, since the ids of a step are
+known at its start, one launch makes the plans of all layers of that many experts and choices.  ``defer_combine``: the
 weighted sum is left to the block (``ExpertRows``), whose residual sum takes it in.
 
 On the device, with nothing read on the host (so a step can be captured in a graph): route -> counting sort of the
@@ -76,7 +77,7 @@ class GroupedMoE(FeedForward):
             raise ValueError("experts named by a table exclude a router's options, a shared expert, identity experts and ungated experts")
         if defer_combine and table is None:
             raise ValueError("only experts of one common weight (named by a table) can leave their sum to the block")
-        self.vocab, self.defer_combine, self.table = None if table is None else int(table), bool(defer_combine), None
+        self.vocab, self.defer_combine, self.tables = None if table is None else int(table), bool(defer_combine), None
         self.expert_kind, self.act, self.weight_on_input, self.shared_gate = expert, act, weight_on == "input", shared_gate
         self.score, self.has_correction, self.identity, self.routed = score, bool(correction), int(identity), routed
         self.d_model, self.hidden, self.experts, self.top = int(d_model), int(hidden), int(experts), int(top)
@@ -132,7 +133,17 @@ class GroupedMoE(FeedForward):
         low, high = int(table.min()), int(table.max())
         if low < 0 or high >= self.experts:
             raise ValueError(f"{self.prefix}.{self.names['table']}: experts {low} .. {high} are named, the layer has {self.experts}")
-        self.table = table.to(torch.int32).contiguous()
+        self.tables, self.table_index = table.to(torch.int32).contiguous()[None], 0
+
+    def link(self, parts):
+        """The tables of all layers of equal sizes lie in one tensor, made by the first of them."""
+        if self.vocab is None:
+            return
+        alike = [p for p in parts if isinstance(p, GroupedMoE) and p.vocab is not None and (p.vocab, p.experts, p.top) == (self.vocab, self.experts, self.top)]
+        if alike[0] is self and len(alike) > 1:
+            tables = torch.cat([p.tables[p.table_index:p.table_index + 1] for p in alike]).contiguous()
+            for i, p in enumerate(alike):
+                p.tables, p.table_index = tables, i
 
     def _load_router(self, params):
         self.w_router = params[self.names["router"]].contiguous()
@@ -173,7 +184,11 @@ class GroupedMoE(FeedForward):
 
     def _table_forward(self, x: torch.Tensor, ctx: StepContext):
         ops, T = self.ops, x.shape[0]
-        plan = ops.moe_plan_table(self.table, ctx.token_ids, self.experts)
+        key = ("expert plans", self.tables.data_ptr())
+        plans = ctx.step_cache.get(key)
+        if plans is None:
+            plans = ctx.step_cache[key] = ops.moe_plan_table(self.tables, ctx.token_ids, self.experts)
+        plan = plans[self.table_index]
         act = ops.grouped_glu(x, self.w_gu, plan, self.top, self.hidden, self.alpha, self.limit or 0.0, self.shift)
         y = ops.grouped_linear(act, self.w_down, plan, out_dtype=torch.float32)
         experts = ExpertRows(y, plan, self.top, 1.0 / self.top)
