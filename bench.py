@@ -632,7 +632,7 @@ def run_design(args, pk):
             saved, eng.stepper.graph_batch_sizes = eng.stepper.graph_batch_sizes, []
 
             def decode_once():
-                eng.stepper.step([StepEntry(rid, ctx - 1, [7], [0]) for rid in rids])
+                eng.stepper.step([StepEntry(rid, ctx - 1, [7 + 11 * i], [0]) for i, rid in enumerate(rids)])     # (different tokens: experts may go by the id)
 
             d_ops = time_ops(eng, decode_once, pk, [(ctx, 1)] * batch, window)
             eng.stepper.graph_batch_sizes = saved

@@ -187,6 +187,28 @@ def test_greedy_generation_through_the_scheduler(graphs):
     assert eng.generate(prompts, SamplingParams(max_new_tokens=14, greedy=True)) == want
 
 
+@pytest.mark.parametrize("graphs", [False, True])
+def test_two_streams_change_nothing(ops, graphs):
+    """Small steps run a layer's feed-forward beside its attention; the same steps on one stream give the same bits, eagerly and from
+    captured graphs, also where steps of either kind alternate."""
+    cfg = dict(FOK_C, max_seq_len=256)
+    w = weights_for(cfg, 19)
+    prompts = [list(range(3, 80)), [4, 4, 9], list(range(50, 57))]
+    runs = {}
+    saved = ops.branch_max_tokens
+    try:
+        for limit in (0, 20, 64):
+            ops.branch_max_tokens = limit
+            eng = engine_for(cfg, w, "float32", pages=60, budget=40, graphs=graphs)
+            assert eng.ops is ops
+            runs[limit] = (tu.run_steps(eng, tu.mixed(requests(cfg, [60, 90, 5], 6))), eng.generate(prompts, SamplingParams(max_new_tokens=20, greedy=True)))
+    finally:
+        ops.branch_max_tokens = saved
+    for limit in (20, 64):
+        assert runs[limit][1] == runs[0][1]
+        assert all(torch.equal(row, runs[limit][0][key]) for key, row in runs[0][0].items())
+
+
 def test_command_line_and_trace_runner_with_a_model_folder(tmp_path):
     """A folder written in the random-weights mode (bfloat16 on disk), generated from by the command line and replayed by the
     trace runner: the architecture is picked from config.json by both."""
@@ -464,6 +486,31 @@ def test_table_experts_alone(ops, dtype, T, experts, top):
             assert ops.residual_sum(out, None, experts=(y.rows, y.plan, y.top, y.weight)) is None
             y = out
         assert rel(y, pf.table_experts(x.double(), w, "", f, toks)) < (2e-5 if dtype == "float32" else 2e-2)
+
+
+@pytest.mark.parametrize("few", [0, 1, 2])
+@pytest.mark.parametrize("T,experts,top,width,ff", [(1, 3, 1, 8, 8), (9, 4, 2, 56, 24), (40, 3, 3, 200, 72), (33, 2, 1, 1032, 136), (70, 20, 5, 128, 40)])
+def test_grouped_products_in_every_form(ops, monkeypatch, few, T, experts, top, width, ff):
+    """The library's, and weights streamed once for eight or sixteen rows at a time: gated and plain, either output, tiles of a single row
+    and of more than sixteen, widths that leave warps without a share of the sum, an activation behind a row's weight."""
+    monkeypatch.setattr(ops, "_grouped_few", lambda x, plan: few)
+    g = torch.Generator().manual_seed(T)
+    r = lambda *s: (torch.randn(s, generator=g) / s[-1] ** 0.5).to(torch.bfloat16)
+    w_gu, w_down, x = r(experts, 2 * ff, width), r(experts, width, ff), torch.randn(T, width, generator=g).to(torch.bfloat16)
+    table = torch.rand(1, 30, experts, generator=g).argsort(-1)[..., :top].to(torch.int32).contiguous()
+    ids = torch.randint(0, 30, (T,), generator=g).to(torch.int32)
+    plan = ops.moe_plan_table(table.to(DEV), ids.to(DEV), experts)[0]
+    pair = plan["pair_of_pos"].cpu().long()
+    tok, ex = pair // top, table[0][ids.long()].reshape(-1)[pair].long()
+    gu = torch.einsum("pd,pfd->pf", x.double()[tok], w_gu.double()[ex])
+    act = ops.grouped_glu(x.to(DEV), w_gu.to(DEV), plan, top, ff)
+    assert rel(act, pf.silu(gu[:, :ff]) * gu[:, ff:]) < 2e-2
+    y = torch.einsum("pf,pdf->pd", act.double().cpu(), w_down.double()[ex])
+    for out_dtype in (torch.float32, torch.bfloat16):
+        assert rel(ops.grouped_linear(act, w_down.to(DEV), plan, out_dtype=out_dtype), y) < 1e-2
+    scale = torch.rand(T, top, generator=g)
+    up = ops.grouped_act(x.to(DEV), w_gu.to(DEV), plan, top, "relu2", row_scale=scale.to(DEV))
+    assert rel(up, torch.relu(gu * scale.reshape(-1)[pair][:, None].double()) ** 2) < 2e-2
 
 
 @pytest.mark.parametrize("T", [1, 63, 700])

@@ -246,7 +246,7 @@ grouped_gemm_kernel(const T* __restrict__ A, long long lda, const int* __restric
     }
 }
 
-// ---- few rows (decode steps): every tile's weights are streamed once.  A warp owns GV_ROWS weight rows of the tile's expert,
+// ---- few rows (decode steps): every tile's weights are streamed once.  32-bit: a warp owns GV_ROWS weight rows of the tile's expert,
 // its lanes walk K in 16-byte steps, the tile's activation rows (a few, read by every warp) come through the cache MT at a
 // time; lane-partial sums are added by shuffles in a fixed order.  K a multiple of the vector, rows 16-byte aligned.
 constexpr int GV_WARPS = 8, GV_ROWS = 4;
@@ -329,6 +329,120 @@ grouped_gemv_kernel(const T* __restrict__ A, long long lda, const int* __restric
                 for (int r = 0; r < GV_ROWS; ++r)
                     if (m0 + m < rows && n0 + r < N)
                         C[(size_t)(r0 + m0 + m) * ldc + n0 + r] = from_f32<TO>(row_act(ra, acc[m][r], row_scale_of(ra, r0 + m0 + m)));
+        }
+    }
+}
+
+// The same in bfloat16 on the tensor cores: the weight rows take the product's 16-row side and the tile's activation rows, eight at a
+// time (MT sets of eight for tiles that are likely to hold more), its 8-column side.  A CTA owns 16 weight rows of the tile's expert (gated: 16 gate rows and the 16 up rows that go with
+// them); its four warps split K, every lane streams 16-byte pieces of two rows per set straight into mma fragments (the order of k
+// inside a sum is free, so a piece of eight k feeds two steps and both operands agree on which k sits where), two buffers of U
+// pieces in flight; the warps' sums are added in a fixed order.
+__device__ __forceinline__ uint4 ld_stream16(const void* p) {
+    uint4 v;
+    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];\n" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+    return v;
+}
+__device__ __forceinline__ void mma_m16n8k16(float (&c)[4], unsigned a0, unsigned a1, unsigned a2, unsigned a3, unsigned b0, unsigned b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+template <typename TO, int SETS, int U, int MT>
+__global__ void __launch_bounds__(128)
+grouped_skinny_kernel(const __nv_bfloat16* __restrict__ A, long long lda, const int* __restrict__ row_of, int row_div,
+                      const __nv_bfloat16* __restrict__ W, long long w_stride, long long ldw, TO* __restrict__ C, long long ldc,
+                      const int* __restrict__ tiles, const int* __restrict__ meta, int N, int K, GluConst glu, RowAct ra) {
+    __shared__ float red[4][SETS][MT][32][4];
+    TTIE_PDL_ENTRY();
+    const int tile = blockIdx.y;
+    if (tile >= meta[0]) return;
+    const int expert = tiles[4 * tile], r0 = tiles[4 * tile + 1], rows = tiles[4 * tile + 2];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane >> 2, q = lane & 3;
+    const int n0 = blockIdx.x * 16, limit = SETS == 2 ? glu.F : N;   // (gated: set 1 holds the up rows, glu.F further down)
+    const int kq = (K + 127) / 128 * 32;
+    const int k_begin = warp * kq, k_end = min(K, k_begin + kq);
+    const bool ok_a = n0 + r < limit, ok_b = n0 + r + 8 < limit;
+    const __nv_bfloat16* wrow[SETS][2];
+#pragma unroll
+    for (int s = 0; s < SETS; ++s) {
+        const __nv_bfloat16* base = W + (size_t)expert * w_stride + (size_t)(s ? glu.F : 0) * ldw;
+        wrow[s][0] = base + (size_t)(ok_a ? n0 + r : 0) * ldw;
+        wrow[s][1] = base + (size_t)(ok_b ? n0 + r + 8 : 0) * ldw;
+    }
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    for (int m0 = 0; m0 < rows; m0 += 8 * MT) {
+        bool ok_x[MT];
+        const __nv_bfloat16* xrow[MT];
+#pragma unroll
+        for (int j = 0; j < MT; ++j) {
+            ok_x[j] = m0 + 8 * j + r < rows;
+            const int pos_x = r0 + (ok_x[j] ? m0 + 8 * j + r : 0);
+            xrow[j] = A + (size_t)(row_of ? row_of[pos_x] / row_div : pos_x) * lda;
+        }
+        float acc[SETS][MT][4];
+#pragma unroll
+        for (int s = 0; s < SETS; ++s)
+#pragma unroll
+            for (int j = 0; j < MT; ++j) { acc[s][j][0] = acc[s][j][1] = acc[s][j][2] = acc[s][j][3] = 0.f; }
+        uint4 wA[U][SETS][2], xA[U][MT], wB[U][SETS][2], xB[U][MT];
+        auto load = [&](int k0, uint4 (&wv)[U][SETS][2], uint4 (&xv)[U][MT]) {  // (past k_end: zeros)
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                const int kk = k0 + 32 * u + 8 * q;
+                const bool ok = kk < k_end;
+#pragma unroll
+                for (int s = 0; s < SETS; ++s) {
+                    wv[u][s][0] = (ok && ok_a) ? ld_stream16(wrow[s][0] + kk) : zero;
+                    wv[u][s][1] = (ok && ok_b) ? ld_stream16(wrow[s][1] + kk) : zero;
+                }
+#pragma unroll
+                for (int j = 0; j < MT; ++j) xv[u][j] = (ok && ok_x[j]) ? __ldg(reinterpret_cast<const uint4*>(xrow[j] + kk)) : zero;
+            }
+        };
+        auto compute = [&](const uint4 (&wv)[U][SETS][2], const uint4 (&xv)[U][MT]) {
+#pragma unroll
+            for (int u = 0; u < U; ++u)
+#pragma unroll
+                for (int s = 0; s < SETS; ++s)
+#pragma unroll
+                    for (int j = 0; j < MT; ++j) {
+                        mma_m16n8k16(acc[s][j], wv[u][s][0].x, wv[u][s][1].x, wv[u][s][0].y, wv[u][s][1].y, xv[u][j].x, xv[u][j].y);
+                        mma_m16n8k16(acc[s][j], wv[u][s][0].z, wv[u][s][1].z, wv[u][s][0].w, wv[u][s][1].w, xv[u][j].z, xv[u][j].w);
+                    }
+        };
+        load(k_begin, wA, xA);
+        load(k_begin + 32 * U, wB, xB);
+        for (int k0 = k_begin; k0 < k_end; k0 += 64 * U) {
+            compute(wA, xA);
+            if (k0 + 64 * U < k_end) load(k0 + 64 * U, wA, xA);
+            if (k0 + 32 * U < k_end) {
+                compute(wB, xB);
+                if (k0 + 96 * U < k_end) load(k0 + 96 * U, wB, xB);
+            }
+        }
+        if (m0) __syncthreads();                                     // (the sums of the rows before have been read)
+#pragma unroll
+        for (int s = 0; s < SETS; ++s)
+#pragma unroll
+            for (int j = 0; j < MT; ++j)
+#pragma unroll
+                for (int c = 0; c < 4; ++c) red[warp][s][j][lane][c] = acc[s][j][c];
+        __syncthreads();
+        const int c = warp, n = n0 + r + 8 * (c >> 1);               // thread (lane, c) finishes element c of `lane`
+#pragma unroll
+        for (int j = 0; j < MT; ++j) {
+            const int m = m0 + 8 * j + 2 * q + (c & 1);
+            if (m >= rows || n >= limit) continue;
+            float v[SETS];
+#pragma unroll
+            for (int s = 0; s < SETS; ++s) v[s] = ((red[0][s][j][lane][c] + red[1][s][j][lane][c]) + red[2][s][j][lane][c]) + red[3][s][j][lane][c];
+            float out;
+            if (SETS == 2) {
+                float g = v[0], u = v[SETS - 1];
+                if (glu.limit > 0.f) { g = fminf(g, glu.limit); u = fminf(fmaxf(u, -glu.limit), glu.limit); }
+                out = g / (1.0f + expf(-glu.alpha * g)) * (u + glu.shift);
+            } else out = row_act(ra, v[0], row_scale_of(ra, r0 + m));
+            C[(size_t)(r0 + m) * ldc + n] = from_f32<TO>(out);
         }
     }
 }
@@ -498,6 +612,7 @@ extern "C" int ttie_moe_plan_table(const int* table, int layers, long long out_s
     return launch_plan({nullptr, table, token_ids, top, vocab, E}, layers, out_stride, T * top, E, E, max_tiles, offsets, pos_of_pair, pair_of_pos, tiles, meta, (cudaStream_t)stream);
 }
 
+// few_rows: 0 tiles of 64 rows; 1 every tile's weights streamed for its rows, 16-bit operands eight rows at a time; 2 sixteen at a time
 // act, row_scale, scale_of: an activation behind an ungated product, see RowAct (act 0 and row_scale null: the plain product)
 extern "C" int ttie_grouped_gemm_act(const void* A, long long lda, const int* row_of, int row_div, const void* W, long long w_stride,
                                      long long ldw, void* C, long long ldc, const int* tiles, const int* meta, int max_tiles, int N, int K,
@@ -525,12 +640,25 @@ extern "C" int ttie_grouped_gemm_act(const void* A, long long lda, const int* ro
     if (few_rows && K % vn == 0 && lda % vn == 0 && ldw % vn == 0 && w_stride % vn == 0 && (((uintptr_t)A | (uintptr_t)W) & 15) == 0 && esz) {
         if (glu_F > 0 && N != 2 * glu_F) TTIE_FAIL("grouped_gemm: a gated epilogue of width %d on a matrix of %d rows", glu_F, N);
         const GluConst glu{glu_F, glu_alpha, glu_limit, glu_shift};
+        if (dtype == kBF16) {
+            const dim3 gs(ceil_div(glu_F > 0 ? glu_F : N, 16), max_tiles);
+#define GS(TO, SETS, U) do { if (few_rows > 1) GSM(TO, SETS, U, 2); else GSM(TO, SETS, U, 1); } while (0)
+#define GSM(TO, SETS, U, MT) TTIE_LAUNCH((grouped_skinny_kernel<TO, SETS, U, MT>), gs, 128, 0, s, (const __nv_bfloat16*)A, lda, row_of, row_div > 0 ? row_div : 1, \
+                                    (const __nv_bfloat16*)W, w_stride, ldw, (TO*)C, ldc, tiles, meta, N, K, glu, ra)
+            if (glu_F > 0 && out_dtype == kBF16) GS(__nv_bfloat16, 2, 2);
+            else if (glu_F > 0) TTIE_FAIL("grouped_gemm: a gated epilogue of 16-bit operands with output dtype %d", out_dtype);
+            else if (out_dtype == kBF16) GS(__nv_bfloat16, 1, 2);
+            else if (out_dtype == kF32) GS(float, 1, 2);
+            else TTIE_FAIL("grouped_gemm: operand dtype %d with output dtype %d", dtype, out_dtype);
+#undef GS
+#undef GSM
+            TTIE_CHECK_LAUNCH("grouped_gemm (few rows)");
+            return 0;
+        }
         const dim3 g(glu_F > 0 ? ceil_div(glu_F, GV_WARPS * GV_ROWS / 2) : ceil_div(N, GV_WARPS * GV_ROWS), max_tiles);
 #define GV(TT, TO) TTIE_LAUNCH((grouped_gemv_kernel<TT, TO, 4>), g, GV_WARPS * 32, 0, s, (const TT*)A, lda, row_of, row_div > 0 ? row_div : 1, (const TT*)W, \
                                w_stride, ldw, (TO*)C, ldc, tiles, meta, N, K, glu, ra)
         if (dtype == kF32 && out_dtype == kF32) GV(float, float);
-        else if (dtype == kBF16 && out_dtype == kBF16) GV(__nv_bfloat16, __nv_bfloat16);
-        else if (dtype == kBF16 && out_dtype == kF32) GV(__nv_bfloat16, float);
         else TTIE_FAIL("grouped_gemm: operand dtype %d with output dtype %d", dtype, out_dtype);
 #undef GV
         TTIE_CHECK_LAUNCH("grouped_gemm (few rows)");

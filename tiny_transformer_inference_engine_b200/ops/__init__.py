@@ -1566,8 +1566,20 @@ class CudaOps:
         self.launches += 1
         return plans
 
-    grouped_few_rows = 48                   # (token, choice) pairs up to which the grouped product streams every tile's weights once (16 experts of [1024, 1024] to
-                                            # [4096, 4096]: ahead of the library up to 32 to 48 pairs, level or behind at 64)
+    # (token, choice) pairs up to which the grouped product streams every tile's weights once; in bfloat16 also up to so many pairs
+    # per expert.  (16 experts of [4096, 4096] and [4096, 2048]: 128 us against the library's 190 at 64 pairs, 140 against 200 at
+    # 192, level at 256; 64 experts of [1536, 2048]: 103 against 148 at 384 pairs.)
+    grouped_few_rows = {torch.float32: 64, torch.bfloat16: 32}
+    grouped_rows_per_expert = 14
+
+    def _grouped_few(self, x, plan):
+        """0: tiles of 64 rows; 1 or 2: the grouped product streams every tile's weights once, eight or sixteen rows at a time."""
+        pairs, experts = plan["pairs"], max(1, plan["real_experts"])
+        if x.dtype == torch.float32:
+            return 1 if pairs <= self.grouped_few_rows[x.dtype] else 0
+        if pairs > max(self.grouped_few_rows[x.dtype], self.grouped_rows_per_expert * experts):
+            return 0
+        return 2 if pairs > 6 * experts else 1
 
     def _library_grouped(self, x, w, plan, gather_div):
         """The library's grouped product (bfloat16, many rows): rows gathered into expert order, then one call whose group
@@ -1616,14 +1628,14 @@ class CudaOps:
     def grouped_glu(self, x, w_gu, plan, gather_div, hidden, alpha=1.0, limit=0.0, shift=0.0):
         """The experts' gate/up products over rows sorted by expert, then the gated unit: [pairs, hidden].  Few rows: one
         kernel (the unit in the weight-streaming product's epilogue); many: the grouped product and the activation kernel."""
-        few = plan["pairs"] <= self.grouped_few_rows
+        few = self._grouped_few(x, plan)
         E, N, K = w_gu.shape
         vn = 4 if x.dtype == torch.float32 else 8
         if few and K % vn == 0 and x.stride(0) % vn == 0:
             out = torch.empty((plan["pairs"], hidden), dtype=x.dtype, device=x.device)
             self._check(self.lib.ttie_grouped_gemm(_ptr(x), x.stride(0), _ptr(plan["pair_of_pos"]) if gather_div else None, int(gather_div),
                                                    _ptr(w_gu), w_gu.stride(0), w_gu.stride(1), _ptr(out), hidden, _ptr(plan["tiles"]),
-                                                   _ptr(plan["meta"]), plan["max_tiles"], N, K, self._dt(x), self._dt(out), 1, int(hidden),
+                                                   _ptr(plan["meta"]), plan["max_tiles"], N, K, self._dt(x), self._dt(out), few, int(hidden),
                                                    float(alpha), float(limit or 0.0), float(shift), self._stream(x)), "grouped_gemm (gated)")
             self.launches += 1
             return out
@@ -1639,7 +1651,7 @@ class CudaOps:
         activation is the product's epilogue; many rows in bfloat16: the library's grouped product, then one pass in place."""
         E, N, K = w_up.shape
         code = self._ROW_ACTS[act]
-        few = plan["pairs"] <= self.grouped_few_rows
+        few = self._grouped_few(x, plan)
         scale_of = plan["pair_of_pos"] if row_scale is not None else None
         if not few and x.dtype == torch.bfloat16:
             out = self._library_grouped(x, w_up, plan, gather_div)
@@ -1652,7 +1664,7 @@ class CudaOps:
         out = torch.empty((plan["pairs"], N), dtype=x.dtype, device=x.device)
         self._check(self.lib.ttie_grouped_gemm_act(_ptr(x), x.stride(0), _ptr(plan["pair_of_pos"]) if gather_div else None, int(gather_div),
                                                    _ptr(w_up), w_up.stride(0), w_up.stride(1), _ptr(out), N, _ptr(plan["tiles"]),
-                                                   _ptr(plan["meta"]), plan["max_tiles"], N, K, self._dt(x), self._dt(out), 1 if few else 0,
+                                                   _ptr(plan["meta"]), plan["max_tiles"], N, K, self._dt(x), self._dt(out), few,
                                                    0, 1.0, 0.0, 0.0, code, _ptr(row_scale), _ptr(scale_of), self._stream(x)),
                     "grouped_gemm (activation)")
         self.launches += 1
@@ -1664,7 +1676,7 @@ class CudaOps:
         weights once; many rows in bfloat16: the library's grouped product (its result is bfloat16 whatever ``out_dtype``
         asks: it has no wider output); else (float32) FFMA tiles."""
         E, N, K = w.shape
-        few = plan["pairs"] <= self.grouped_few_rows
+        few = self._grouped_few(x, plan)
         if not few and x.dtype == torch.bfloat16:
             out = self._library_grouped(x, w, plan, gather_div)
             if out is not None:
@@ -1672,7 +1684,7 @@ class CudaOps:
         out = torch.empty((plan["pairs"], N), dtype=out_dtype or x.dtype, device=x.device)
         self._check(self.lib.ttie_grouped_gemm(_ptr(x), x.stride(0), _ptr(plan["pair_of_pos"]) if gather_div else None, int(gather_div),
                                                _ptr(w), w.stride(0), w.stride(1), _ptr(out), N, _ptr(plan["tiles"]), _ptr(plan["meta"]),
-                                               plan["max_tiles"], N, K, self._dt(x), self._dt(out), 1 if few else 0, 0, 1.0, 0.0, 0.0,
+                                               plan["max_tiles"], N, K, self._dt(x), self._dt(out), few, 0, 1.0, 0.0, 0.0,
                                                self._stream(x)), "grouped_gemm")
         self.launches += 1
         return out
